@@ -90,7 +90,8 @@ class PagedCache:
         for n in self.requests:
             self.roles.setdefault(n.run, []).append(n.role)
         h = host()
-        self.book = h.CacheManager([h.GroupSpec(g.page_size, g.num_pages, g.request.window, g.request.keep_first)
+        self.book = h.CacheManager([h.GroupSpec(g.page_size, g.num_pages, g.request.window, g.request.keep_first,
+                                                  g.request.chunk)
                                     for g in self.groups], self.max_seqs, self.max_pages_per_seq)
         self.state: Dict[Tuple[int, str], torch.Tensor] = {}
         if allocate:
@@ -177,12 +178,15 @@ class PagedCache:
 
     def kv_bytes_read(self, cached_tokens: float) -> float:
         """Bytes of keys and values that one token reads of a request with `cached_tokens` tokens: every group's
-        rows, a group with a window no more than the window and its kept first keys."""
+        rows, a group with a window no more than the window and its kept first keys, a group in chunks no more than
+        what its token's chunk holds so far."""
         es = torch.empty((), dtype=self.dtype).element_size()
         total = 0.0
         for g in self.groups:
             r = g.request
             seen = min(cached_tokens, r.window + r.keep_first) if r.window > 0 else cached_tokens
+            if r.chunk > 0:
+                seen = cached_tokens % r.chunk + 1
             total += g.bytes_per_token * seen
         return total * es
 
@@ -190,5 +194,5 @@ class PagedCache:
         return {f"group{g}": dict(pages=grp.num_pages, in_use=self.book.pages_in_use(g),
                                   high_water=self.book.high_water(g),
                                   allocations=self.book.total_allocations(g),
-                                  window=grp.request.window)
+                                  window=grp.request.window, chunk=grp.request.chunk)
                 for g, grp in enumerate(self.groups)}

@@ -18,3 +18,6 @@ __all__.append("TizodraConfig")
 from .fokisun import FokisunConfig  # noqa: E402
 
 __all__.append("FokisunConfig")
+from .vatazen import VatazenConfig  # noqa: E402
+
+__all__.append("VatazenConfig")

@@ -8,6 +8,7 @@ from __future__ import annotations
 
 import json
 import os
+from typing import Callable, Optional
 
 
 class ConfigError(ValueError):
@@ -63,3 +64,22 @@ def get_bool(raw: dict, key: str, default: bool) -> bool:
     if not isinstance(v, bool):
         raise ConfigError(f"config.json: `{key}` must be true or false, got {v!r}")
     return v
+
+
+def get_object(raw: dict, key: str, required: bool = True) -> Optional[dict]:
+    v = raw.get(key)
+    if v is None:
+        if required:
+            raise ConfigError(f"config.json: required key `{key}` is missing")
+        return None
+    if not isinstance(v, dict):
+        raise ConfigError(f"config.json: `{key}` must be an object, got {v!r}")
+    return v
+
+
+def named(read: Callable, where: str):
+    """Run a reader of a nested object and put the object's place in front of its complaint."""
+    try:
+        return read()
+    except ConfigError as e:
+        raise ConfigError(str(e).replace("config.json: ", f"config.json: {where}", 1)) from None

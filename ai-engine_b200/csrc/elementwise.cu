@@ -4,11 +4,11 @@
 #include "common.cuh"
 
 // ---------------------------------------------------------------------------
-// x[t, :] = float(E[ids[t], :])        (crates/ai-engine-runtime/src/arch/embedding.rs:14-20)
+// x[t, :] = float(E[ids[t], :]) * scale        (crates/ai-engine-runtime/src/arch/embedding.rs:14-20)
 // ---------------------------------------------------------------------------
 template <typename W>
 __global__ void embed_gather_kernel(const int* __restrict__ ids, const W* __restrict__ table,
-                                    float* __restrict__ x, int D, int vocab, unsigned* err) {
+                                    float* __restrict__ x, int D, int vocab, float scale, unsigned* err) {
     const int t = blockIdx.x;
     int id = ids[t];
     if (id < 0 || id >= vocab) {
@@ -17,12 +17,12 @@ __global__ void embed_gather_kernel(const int* __restrict__ ids, const W* __rest
         return;
     }
     const W* row = table + (size_t)id * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) x[(size_t)t * D + i] = to_f32<W>(row[i]);
+    for (int i = threadIdx.x; i < D; i += blockDim.x) x[(size_t)t * D + i] = to_f32<W>(row[i]) * scale;
 }
 
 // bf16 table, D a multiple of 8: 16-byte loads, two float4 stores per thread
 __global__ void embed_gather_vec_kernel(const int* __restrict__ ids, const bf16* __restrict__ table,
-                                        float* __restrict__ x, int D, int vocab, unsigned* err) {
+                                        float* __restrict__ x, int D, int vocab, float scale, unsigned* err) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -36,8 +36,8 @@ __global__ void embed_gather_vec_kernel(const int* __restrict__ ids, const bf16*
         if (ok) {
             const uint4 raw = row[i];
             const bf16* e = reinterpret_cast<const bf16*>(&raw);
-            a = make_float4(__bfloat162float(e[0]), __bfloat162float(e[1]), __bfloat162float(e[2]), __bfloat162float(e[3]));
-            b = make_float4(__bfloat162float(e[4]), __bfloat162float(e[5]), __bfloat162float(e[6]), __bfloat162float(e[7]));
+            a = make_float4(__bfloat162float(e[0]) * scale, __bfloat162float(e[1]) * scale, __bfloat162float(e[2]) * scale, __bfloat162float(e[3]) * scale);
+            b = make_float4(__bfloat162float(e[4]) * scale, __bfloat162float(e[5]) * scale, __bfloat162float(e[6]) * scale, __bfloat162float(e[7]) * scale);
         }
         dst[2 * i] = a;
         dst[2 * i + 1] = b;
@@ -45,14 +45,14 @@ __global__ void embed_gather_vec_kernel(const int* __restrict__ ids, const bf16*
 }
 
 extern "C" int aie_embed_gather(const int* ids, const void* table, int table_dtype, float* x,
-                                int T, int D, int vocab, unsigned* err, cudaStream_t stream) {
+                                int T, int D, int vocab, float scale, unsigned* err, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (table_dtype == AIE_F32)
-        embed_gather_kernel<float><<<T, 256, 0, stream>>>(ids, (const float*)table, x, D, vocab, err);
+        embed_gather_kernel<float><<<T, 256, 0, stream>>>(ids, (const float*)table, x, D, vocab, scale, err);
     else if (table_dtype == AIE_BF16 && D % 8 == 0)
-        launch_pdl(embed_gather_vec_kernel, dim3(T), dim3(D >= 4096 ? 512 : 128), 0, stream, ids, (const bf16*)table, x, D, vocab, err);
+        launch_pdl(embed_gather_vec_kernel, dim3(T), dim3(D >= 4096 ? 512 : 128), 0, stream, ids, (const bf16*)table, x, D, vocab, scale, err);
     else if (table_dtype == AIE_BF16)
-        embed_gather_kernel<bf16><<<T, 256, 0, stream>>>(ids, (const bf16*)table, x, D, vocab, err);
+        embed_gather_kernel<bf16><<<T, 256, 0, stream>>>(ids, (const bf16*)table, x, D, vocab, scale, err);
     else
         return AIE_BAD_ARG;
     AIE_LAUNCH_CHECK();

@@ -28,14 +28,16 @@ PYBIND11_MODULE(_aie_host, m) {
         .def("release", &PagePool::release);
 
     py::class_<GroupSpec>(m, "GroupSpec")
-        .def(py::init([](int page_size, int num_pages, int window, int keep_first) {
+        .def(py::init([](int page_size, int num_pages, int window, int keep_first, int chunk) {
                  GroupSpec g; g.page_size = page_size; g.num_pages = num_pages; g.window = window;
-                 g.keep_first = keep_first; return g;
-             }), py::arg("page_size"), py::arg("num_pages"), py::arg("window") = 0, py::arg("keep_first") = 0)
+                 g.keep_first = keep_first; g.chunk = chunk; return g;
+             }), py::arg("page_size"), py::arg("num_pages"), py::arg("window") = 0, py::arg("keep_first") = 0,
+             py::arg("chunk") = 0)
         .def_readwrite("page_size", &GroupSpec::page_size)
         .def_readwrite("num_pages", &GroupSpec::num_pages)
         .def_readwrite("window", &GroupSpec::window)
-        .def_readwrite("keep_first", &GroupSpec::keep_first);
+        .def_readwrite("keep_first", &GroupSpec::keep_first)
+        .def_readwrite("chunk", &GroupSpec::chunk);
 
     py::class_<CacheManager>(m, "CacheManager")
         .def(py::init<std::vector<GroupSpec>, int, int>(), py::arg("groups"), py::arg("max_seqs"), py::arg("max_pages_per_seq"))

@@ -73,6 +73,12 @@ struct GroupSpec {
     int num_pages = 0;    // pages of this group's pool
     int window = 0;       // 0: every key is kept; w > 0: a query at p reads keys in (p - w, p]
     int keep_first = 0;   // with a window: keys [0, keep_first) stay readable for every later query
+    int chunk = 0;        // c > 0: a query at p reads keys in [p / c * c, p] (a window and a chunk exclude each other)
+    // first key that a query at `pos` or later can read (kept first keys aside)
+    int first_key(int pos) const {
+        if (chunk > 0) return pos / chunk * chunk;
+        return window > 0 ? std::max(0, pos - window + 1) : 0;
+    }
 };
 
 struct SeqTable {
@@ -91,6 +97,9 @@ class CacheManager {
             if (g.page_size <= 0) throw std::invalid_argument("CacheManager: page_size must be positive");
             if (g.window < 0) throw std::invalid_argument("CacheManager: negative window");
             if (g.keep_first < 0) throw std::invalid_argument("CacheManager: negative keep_first");
+            if (g.chunk < 0) throw std::invalid_argument("CacheManager: negative chunk");
+            if (g.chunk > 0 && (g.window > 0 || g.keep_first > 0))
+                throw std::invalid_argument("CacheManager: a group has a window or a chunk, not both");
             pools_.emplace_back(g.num_pages);
             tables_.emplace_back(max_seqs);
         }
@@ -149,14 +158,13 @@ class CacheManager {
     }
 
     // `computed` tokens are in the cache and every later query sits at >= computed:
-    // window groups give back the pages that no later query can read.
+    // window and chunk groups give back the pages that no later query can read.
     int advance(int slot, int computed) {
         check_slot(slot);
         int released = 0;
         for (int g = 0; g < num_groups(); ++g) {
-            const int w = groups_[g].window;
-            if (w <= 0) continue;
-            const int first_key = std::max(0, computed - w + 1);
+            if (groups_[g].window <= 0 && groups_[g].chunk <= 0) continue;
+            const int first_key = groups_[g].first_key(computed);
             auto& t = tables_[g][slot];
             const int stop = std::min<int>(first_key / groups_[g].page_size, (int)t.pages.size());
             for (int i = std::max(t.first_live, kept_pages(g)); i < stop; ++i) {
@@ -287,8 +295,8 @@ class Scheduler {
         for (int g = 0; g < cache_->num_groups(); ++g) {
             const auto& gs = cache_->group(g);
             int held = most;
-            if (gs.window > 0)
-                held = std::min(most, gs.window + gs.keep_first + 3 * gs.page_size + std::min(budget_, most));
+            if (gs.window > 0 || gs.chunk > 0)
+                held = std::min(most, gs.window + gs.chunk + gs.keep_first + 3 * gs.page_size + std::min(budget_, most));
             const int pages = (held + gs.page_size - 1) / gs.page_size;
             if (pages > gs.num_pages || (most + gs.page_size - 1) / gs.page_size > cache_->max_pages_per_seq())
                 return "request can never fit the cache (" + std::to_string(most) + " tokens need " + std::to_string(pages) + " pages of group " + std::to_string(g) + ", pool has " + std::to_string(gs.num_pages) + ")";

@@ -9,25 +9,30 @@
 //   query parts (compute dtype, for the folding product), the rotated query parts (float32), and the
 //   normalised c and rotated kr into the token's cache row.  The rotation pairs element 2i with 2i+1 over the
 //   first `rot_dims` elements of the rot-wide part (or, with `halves`, element i with i + rot_dims / 2); the
-//   angle is float(position) * inv_freq[i] in float32.  The latent and the key part may come from a projection
+//   angle is float(position) * inv_freq[i] in float32, and cosine and sine are multiplied by `mag`.  The latent and the key part may come from a projection
 //   of their own (`kv`, rows ld_kv floats apart) when the queries are made by a second product.
 // latent_attention: one block per (token, head); keys in chunks of 128 that start at multiples of 128 of the
 //   absolute key position with a running maximum and sum, so a row's additions depend on its position only.
+//   `sink` (a number per head, or null): the denominator also holds exp(sink[h]), which has no key and no value.
 #include "common.cuh"
 
 #define LAT_CHUNK 128
 
 // element i of a rot-wide vector x after the rotation by `pos`
 __device__ __forceinline__ float latent_rotated(const float* x, int i, int half, int halves, int pos,
-                                                const float* __restrict__ inv_freq) {
+                                                const float* __restrict__ inv_freq, float mag) {
     if (i >= 2 * half) return x[i];
     float sn, cs;
     if (halves) {
         const int j = i < half ? i : i - half;
         sincosf((float)pos * inv_freq[j], &sn, &cs);
+        sn *= mag;
+        cs *= mag;
         return i < half ? x[i] * cs - x[i + half] * sn : x[i] * cs + x[j] * sn;
     }
     sincosf((float)pos * inv_freq[i >> 1], &sn, &cs);
+    sn *= mag;
+    cs *= mag;
     return (i & 1) ? x[i] * cs + x[i - 1] * sn : x[i] * cs - x[i + 1] * sn;
 }
 
@@ -38,7 +43,7 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld, in
                                       float* __restrict__ q_full, C* __restrict__ pages,
                                       const int* __restrict__ positions, const int* __restrict__ token_req,
                                       const int* __restrict__ block_table, int bt_width, int num_pages, int P,
-                                      unsigned* err, const float* __restrict__ kv, int ld_kv, int halves) {
+                                      unsigned* err, const float* __restrict__ kv, int ld_kv, int halves, float mag) {
     __shared__ float red[32];
     const int t = blockIdx.x, tid = threadIdx.x;
     const float* row = proj + (size_t)t * ld;
@@ -52,7 +57,7 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld, in
     for (int e = tid; e < H * rot; e += blockDim.x) {
         const int hh = e / rot, i = e % rot;
         const float* qr = row + hh * dq + d;
-        q_full[((size_t)t * H + hh) * dk + rank + i] = latent_rotated(qr, i, half, halves, pos, inv_freq);
+        q_full[((size_t)t * H + hh) * dk + rank + i] = latent_rotated(qr, i, half, halves, pos, inv_freq, mag);
     }
     if (!has_kv) return;
     const float* z = kv ? kv + (size_t)t * ld_kv : row + H * dq;
@@ -69,20 +74,20 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld, in
     C* dst = pages + ((size_t)page * P + (pos - pidx * P)) * dk;
     for (int i = tid; i < rank; i += blockDim.x) dst[i] = from_f32<C>((z[i] * rinv) * c_weight[i]);
     const float* kr = z + rank;
-    for (int i = tid; i < rot; i += blockDim.x) dst[rank + i] = from_f32<C>(latent_rotated(kr, i, half, halves, pos, inv_freq));
+    for (int i = tid; i < rot; i += blockDim.x) dst[rank + i] = from_f32<C>(latent_rotated(kr, i, half, halves, pos, inv_freq, mag));
 }
 
 extern "C" int aie_latent_prepare(const float* proj, int ld, int T, int H, int d, int rot, int rank, int rot_dims,
                                   int has_kv, const float* c_weight, float eps, const float* inv_freq, void* q_plain,
                                   int q_dtype, float* q_full, void* pages, int cache_dtype, const int* positions,
                                   const int* token_req, const int* block_table, int bt_width, int num_pages, int P,
-                                  unsigned* err, const float* kv, int ld_kv, int halves, cudaStream_t st) {
+                                  unsigned* err, const float* kv, int ld_kv, int halves, float mag, cudaStream_t st) {
     if (T <= 0) return 0;
     if (rot_dims % 2 || rot_dims > rot || H <= 0 || d < 0 || rank <= 0) return AIE_BAD_ARG;
 #define GO(A, C)                                                                                                      \
     latent_prepare_kernel<A, C><<<T, 128, 0, st>>>(proj, ld, H, d, rot, rank, rot_dims, has_kv, c_weight, eps, inv_freq, \
                                                    (A*)q_plain, q_full, (C*)pages, positions, token_req, block_table,  \
-                                                   bt_width, num_pages, P, err, kv, ld_kv, halves)
+                                                   bt_width, num_pages, P, err, kv, ld_kv, halves, mag)
     if (q_dtype == AIE_F32 && cache_dtype == AIE_F32) GO(float, float);
     else if (q_dtype == AIE_BF16 && cache_dtype == AIE_BF16) GO(bf16, bf16);
     else if (q_dtype == AIE_BF16 && cache_dtype == AIE_F32) GO(bf16, float);
@@ -98,7 +103,7 @@ __global__ void __launch_bounds__(LAT_CHUNK)
 latent_attention_kernel(const float* __restrict__ q_full, const C* __restrict__ pages, O* __restrict__ out,
                         const int* __restrict__ positions, const int* __restrict__ token_req,
                         const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int rank,
-                        int dk, int window, float scale, unsigned* err) {
+                        int dk, int window, float scale, const float* __restrict__ sink, unsigned* err) {
     extern __shared__ __align__(16) float sm[];
     float* q_s = sm;                                   // dk (rounded up to even)
     float* p_s = q_s + ((dk + 1) & ~1);                // CHUNK
@@ -112,7 +117,7 @@ latent_attention_kernel(const float* __restrict__ q_full, const C* __restrict__ 
 
     int lo = 0;
     if (window > 0 && pos - window + 1 > 0) lo = pos - window + 1;
-    float m = -INFINITY, l = 0.f;
+    float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;      // the sink opens the running softmax
     float acc[NACC];
 #pragma unroll
     for (int a = 0; a < NACC; ++a) acc[a] = 0.f;
@@ -167,13 +172,13 @@ latent_attention_kernel(const float* __restrict__ q_full, const C* __restrict__ 
 template <typename C, typename O>
 static int latent_go(const float* q_full, const void* pages, void* out, const int* positions, const int* token_req,
                      const int* block_table, int bt_width, int num_pages, int P, int T, int H, int rank, int dk,
-                     int window, float scale, unsigned* err, cudaStream_t st) {
+                     int window, float scale, const float* sink, unsigned* err, cudaStream_t st) {
     const size_t smem = (size_t)(((dk + 1) & ~1) + LAT_CHUNK + 32) * sizeof(float) + LAT_CHUNK * sizeof(long long);
     dim3 grid(T, H);
 #define GO(N)                                                                                                        \
     latent_attention_kernel<C, O, N><<<grid, LAT_CHUNK, smem, st>>>(q_full, (const C*)pages, (O*)out, positions,     \
                                                                     token_req, block_table, bt_width, num_pages, P, \
-                                                                    H, rank, dk, window, scale, err)
+                                                                    H, rank, dk, window, scale, sink, err)
     if (rank <= LAT_CHUNK) GO(1);
     else if (rank <= 2 * LAT_CHUNK) GO(2);
     else if (rank <= 4 * LAT_CHUNK) GO(4);
@@ -185,15 +190,15 @@ static int latent_go(const float* q_full, const void* pages, void* out, const in
 extern "C" int aie_latent_attention(const float* q_full, const void* pages, int cache_dtype, void* out, int out_dtype,
                                     const int* positions, const int* token_req, const int* block_table, int bt_width,
                                     int num_pages, int P, int T, int H, int rank, int dk, int window, float scale,
-                                    unsigned* err, cudaStream_t st) {
+                                    const float* sink, unsigned* err, cudaStream_t st) {
     if (T <= 0) return 0;
     if (rank <= 0 || dk < rank || H <= 0 || H > 65535) return AIE_BAD_ARG;
     if (rank > 8 * LAT_CHUNK || dk > 8192) return AIE_UNSUPPORTED;
     if (cache_dtype == AIE_F32 && out_dtype == AIE_F32)
-        return latent_go<float, float>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, err, st);
+        return latent_go<float, float>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, sink, err, st);
     if (cache_dtype == AIE_BF16 && out_dtype == AIE_BF16)
-        return latent_go<bf16, bf16>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, err, st);
+        return latent_go<bf16, bf16>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, sink, err, st);
     if (cache_dtype == AIE_BF16 && out_dtype == AIE_F32)
-        return latent_go<bf16, float>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, err, st);
+        return latent_go<bf16, float>(q_full, pages, out, positions, token_req, block_table, bt_width, num_pages, P, T, H, rank, dk, window, scale, sink, err, st);
     return AIE_BAD_ARG;
 }

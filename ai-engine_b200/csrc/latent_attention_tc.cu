@@ -13,7 +13,7 @@
 // in shared memory (eight threads a row); O += P V with the latent's columns split over the four warps, V being
 // the first `rank` columns of the same rows (ldmatrix.trans).  Few tokens in a step (decoding) cut each token's
 // chunks into `splits` parts that run as CTAs of their own and leave (maximum, sum, unnormalised output) for a
-// joining kernel.
+// joining kernel.  A sink (exp(sink[h]) in the denominator, no key, no value) opens the running softmax of the first part.
 #include "attention_prefill.cuh"
 
 #define LT_KEYS 64
@@ -26,7 +26,8 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
                            float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ tiles,
                            const int* __restrict__ q_start, const int* __restrict__ q_len,
                            const int* __restrict__ ctx_len, const int* __restrict__ block_table, int bt_width,
-                           int num_pages, int P, int H, int dk, int window, float scale, int splits, unsigned* err) {
+                           int num_pages, int P, int H, int dk, int window, float scale, int splits,
+                           const float* __restrict__ sink, unsigned* err) {
     constexpr int RANK = 4 * CW, NT = CW / 8, THREADS = LT_THREADS * TQ;
     extern __shared__ __align__(16) unsigned char lt_raw[];
     const int SK = dk + 8;                                        // padded row: ldmatrix rows fall on different banks
@@ -69,8 +70,9 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
         }
     }
     if (ltid < LT_ROWS) {
-        m_s[ltid] = -INFINITY;
-        l_s[ltid] = 0.f;
+        const bool leaks = sink && part == 0 && h0 + ltid < H;
+        m_s[ltid] = leaks ? sink[h0 + ltid] : -INFINITY;
+        l_s[ltid] = leaks ? 1.f : 0.f;
     }
     float acc[NT][4];
 #pragma unroll
@@ -259,7 +261,7 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
                                        const int* tiles, int n_tiles, int tq, const int* q_start, const int* q_len,
                                        const int* ctx_len, const int* block_table, int bt_width,
                                        int num_pages, int P, int T, int H, int rank, int dk, int window, float scale,
-                                       int splits, unsigned* err, cudaStream_t st) {
+                                       int splits, const float* sink, unsigned* err, cudaStream_t st) {
     if (T <= 0 || n_tiles <= 0) return 0;
     if (rank < 64 || rank > 512 || rank % 64 || dk % 16 || dk < rank || dk > 1024 || H <= 0) return AIE_UNSUPPORTED;
     if (splits < 1 || splits > 64 || (splits > 1 && (!part_o || !part_ml)) || (tq != 1 && tq != 4)) return AIE_BAD_ARG;
@@ -275,7 +277,7 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
         kern<<<grid, LT_THREADS * TQV, smem, st>>>(q_full, (const bf16*)pages, (bf16*)out, part_o, part_ml, tiles,    \
                                                    q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, H,   \
-                                                   dk, window, scale, splits, err);                                   \
+                                                   dk, window, scale, splits, sink, err);                                   \
     }
 #define GO(CWV)                                                                                                       \
     case CWV:                                                                                                         \

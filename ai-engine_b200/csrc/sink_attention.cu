@@ -6,6 +6,9 @@
 //   out_i = gate[i, h] * sum_j exp(s(i, j)) v_j / (exp(sink[h]) + sum_j exp(s(i, j)))
 //
 // The sink is a term of the denominator that has no key and no value.  Scores, weights and sums are float32.
+// chunk > 0 (without a window): i reads j  iff  j <= i and j / chunk == i / chunk.
+// maps > 1: a key/value head has `maps` keys in front of its one value, a row is [k_0 .. k_(maps-1) | v]; query head h
+// of the H (all maps counted) reads key h % maps of key/value head h / (H / G).
 //
 //   sink_attn_prepare    from a step's fused projection [q | k | v | gate logits] (float32): adds the biases,
 //                        writes q in the compute dtype, divides each head's value by its root mean square
@@ -14,7 +17,9 @@
 //                        [q | k | v] it adds the biases, divides all of q (and all of k) by its root mean square
 //                        over the whole projection, times a weight per element, rotates the first rot_dims
 //                        elements of every head (neighbouring pairs, or halves), mixes the value with another
-//                        layer's value of the same token, and writes q and the cache row [k | v].
+//                        layer's value of the same token, and writes q and the cache row [k | v].  With
+//                        `per_head` every head (and map) of q and k is normed by itself, with one weight of d
+//                        elements for all of them.
 //   sink_attention_plain one block per (query token, head), any sizes up to 256; keys are walked in chunks of
 //                        128 that start at multiples of 128 of the absolute key position, so the order of
 //                        every addition depends on the query's position only.
@@ -105,10 +110,11 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
                            float* __restrict__ v_keep, A* __restrict__ q_out, A* __restrict__ pages,
                            const int* __restrict__ positions, const int* __restrict__ token_req,
                            const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
-                           int e, int write, unsigned* err) {
-    extern __shared__ __align__(16) float np_sm[];     // q (H d) | k (G d) | 32
+                           int e, int maps, int per_head, int write, unsigned* err) {
+    extern __shared__ __align__(16) float np_sm[];     // q (H d) | k (G maps d) | 32
     const int t = blockIdx.x, tid = threadIdx.x;
-    const int nq = H * d, nk = G * d, nv = G * e;
+    const int K = G * maps;                             // keys of a token
+    const int nq = H * d, nk = K * d, nv = G * e;
     float* qs = np_sm;
     float* ks = qs + nq;
     float* red = ks + nk;
@@ -124,9 +130,20 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
         ks[c] = x;
         ssk += x * x;
     }
-    ssq = block_sum(ssq, red);
-    ssk = block_sum(ssk, red);
-    if (q_w) {
+    if (q_w && per_head) {                              // a warp per head
+        __syncthreads();
+        for (int hh = tid >> 5; hh < H + K; hh += blockDim.x >> 5) {
+            float* x = hh < H ? qs + hh * d : ks + (hh - H) * d;
+            const float* wv = hh < H ? q_w : k_w;
+            float ss = 0.f;
+            for (int c = tid & 31; c < d; c += 32) ss += x[c] * x[c];
+            ss = warp_sum(ss);
+            const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+            for (int c = tid & 31; c < d; c += 32) x[c] = (x[c] * inv) * wv[c];
+        }
+    } else if (q_w) {
+        ssq = block_sum(ssq, red);
+        ssk = block_sum(ssk, red);
         const float rq = 1.0f / sqrtf(ssq / (float)nq + eps), rk = 1.0f / sqrtf(ssk / (float)nk + eps);
         for (int c = tid; c < nq; c += blockDim.x) qs[c] = (qs[c] * rq) * q_w[c];
         for (int c = tid; c < nk; c += blockDim.x) ks[c] = (ks[c] * rk) * k_w[c];
@@ -150,20 +167,21 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
     const int page = (pos >= 0 && pidx < bt_width) ? block_table[(size_t)token_req[t] * bt_width + pidx] : -1;
     const bool page_ok = page >= 0 && page < num_pages;
     if (write && !page_ok && tid == 0) atomicOr(err, AIE_DEV_PAGE_OOB);
-    const int w = d + e;
+    const int w = maps * d + e;
     A* base = pages + ((size_t)(page_ok ? page : 0) * G * P + (pos % P)) * w;
     if (write && page_ok) {
-        for (int p = tid; p < G * half; p += blockDim.x) {
-            const int g = p / half, j = p - g * half;
+        for (int p = tid; p < K * half; p += blockDim.x) {
+            const int k = p / half, j = p - k * half;
             int ia, ib;
             float ya, yb;
-            head_pair_rotated(ks + g * d, j, rot_dims, halves, pos, inv_freq, &ia, &ib, &ya, &yb);
-            base[(size_t)g * P * w + ia] = from_f32<A>(ya);
-            base[(size_t)g * P * w + ib] = from_f32<A>(yb);
+            head_pair_rotated(ks + k * d, j, rot_dims, halves, pos, inv_freq, &ia, &ib, &ya, &yb);
+            A* dst = base + (size_t)(k / maps) * P * w + (k % maps) * d;
+            dst[ia] = from_f32<A>(ya);
+            dst[ib] = from_f32<A>(yb);
         }
-        for (int p = tid; p < G * rest; p += blockDim.x) {
-            const int g = p / rest, i = rot_dims + p % rest;
-            base[(size_t)g * P * w + i] = from_f32<A>(ks[g * d + i]);
+        for (int p = tid; p < K * rest; p += blockDim.x) {
+            const int k = p / rest, i = rot_dims + p % rest;
+            base[(size_t)(k / maps) * P * w + (k % maps) * d + i] = from_f32<A>(ks[k * d + i]);
         }
     }
     const float lam = mix_from ? lambda[0] : 0.f;
@@ -173,7 +191,7 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
         if (v_keep) v_keep[(size_t)t * nv + c] = v;
         if (write && page_ok) {
             const int g = c / e;
-            base[(size_t)g * P * w + d + (c - g * e)] = from_f32<A>(v);
+            base[(size_t)g * P * w + maps * d + (c - g * e)] = from_f32<A>(v);
         }
     }
 }
@@ -182,34 +200,41 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
                                        float eps, const float* inv_freq, int rot_dims, int halves, const float* mix_from,
                                        const float* lambda, float* v_keep, void* q_out, void* pages, int dtype,
                                        const int* positions, const int* token_req, const int* block_table, int bt_width,
-                                       int num_pages, int P, int T, int H, int G, int d, int e, int write, unsigned* err,
-                                       cudaStream_t stream) {
+                                       int num_pages, int P, int T, int H, int G, int d, int e, int maps, int per_head,
+                                       int write, unsigned* err, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (maps < 1 || H % maps || (H / maps) % G) return AIE_BAD_ARG;
     if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || rot_dims < 0 || rot_dims > d || rot_dims % 2 ||
         (mix_from && !lambda) || (q_w && !k_w) || (rot_dims > 0 && !inv_freq))
         return AIE_BAD_ARG;
-    const size_t smem = ((size_t)(H + G) * d + 32) * sizeof(float);
-    if (smem > 48 * 1024) return AIE_UNSUPPORTED;
+    const size_t smem = ((size_t)(H + G * maps) * d + 32) * sizeof(float);
+    if (smem > 200 * 1024) return AIE_UNSUPPORTED;
 #define AIE_NAP(A)                                                                                                    \
+    if (smem > 48 * 1024)                                                                                             \
+        cudaFuncSetAttribute(normed_attn_prepare_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
     normed_attn_prepare_kernel<A><<<T, 256, smem, stream>>>(proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, halves, \
                                                            mix_from, lambda, v_keep, (A*)q_out, (A*)pages, positions, \
                                                            token_req, block_table, bt_width, num_pages, P, H, G, d, e, \
-                                                           write, err)
-    if (dtype == AIE_F32) AIE_NAP(float);
-    else if (dtype == AIE_BF16) AIE_NAP(bf16);
-    else return AIE_BAD_ARG;
+                                                           maps, per_head, write, err)
+    if (dtype == AIE_F32) {
+        AIE_NAP(float);
+    } else if (dtype == AIE_BF16) {
+        AIE_NAP(bf16);
+    } else {
+        return AIE_BAD_ARG;
+    }
 #undef AIE_NAP
     AIE_LAUNCH_CHECK();
 }
 
-template <typename A, typename C>
+template <typename A, typename C, typename O>
 __global__ void __launch_bounds__(SA_CHUNK)
-sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages, A* __restrict__ out,
+sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages, O* __restrict__ out,
                             const float* __restrict__ gate, const float* __restrict__ temp,
                             const float* __restrict__ slope, const float* __restrict__ sink,
                             const int* __restrict__ positions, const int* __restrict__ token_req,
                             const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G,
-                            int d, int e, int window, int keep_first, float scale,
+                            int d, int e, int window, int keep_first, int chunk, int maps, float scale,
                             const int* __restrict__ token_list, unsigned* err) {
     extern __shared__ __align__(16) float sm[];
     float* q_s = sm;                                  // d (rounded up to even)
@@ -221,13 +246,14 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
     const int pos = positions[t];
     const int row = token_req[t];
     const int g = h / (H / G);
-    const int w = d + e;
+    const int w = maps * d + e, k_off = (h % maps) * d, v_off = maps * d;
     const float qs = scale * (temp ? temp[h] : 1.f), sl = slope ? slope[h] : 0.f;
     for (int c = tid; c < d; c += blockDim.x) q_s[c] = to_f32<A>(q[((size_t)t * H + h) * d + c]);
     __syncthreads();
 
     int lo = 0;
     if (window > 0 && pos - window + 1 > 0) lo = pos - window + 1;
+    if (chunk > 0) lo = pos / chunk * chunk;
     const int kept = min(keep_first, lo);              // keys [0, kept) are read although the window has passed them
     // the sink opens the running softmax: a weight exp(sink - m) = 1 at m = sink, with no value
     float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f;
@@ -250,7 +276,7 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
                 atomicOr(err, AIE_DEV_PAGE_OOB);
             } else {
                 off = (((long long)page * G + g) * P + (kp % P)) * w;
-                const C* kr = pages + off;
+                const C* kr = pages + off + k_off;
                 float dot = 0.f;
                 for (int c = 0; c < d; ++c) dot += q_s[c] * to_f32<C>(kr[c]);
                 s = dot * qs - sl * (float)(pos - kp);
@@ -272,32 +298,34 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
             const long long o = off_s[j];
             if (o < 0) continue;
             const float pj = p_s[j];
-            if (tid < e) acc0 += pj * to_f32<C>(pages[o + d + tid]);
-            if (tid + SA_CHUNK < e) acc1 += pj * to_f32<C>(pages[o + d + tid + SA_CHUNK]);
+            if (tid < e) acc0 += pj * to_f32<C>(pages[o + v_off + tid]);
+            if (tid + SA_CHUNK < e) acc1 += pj * to_f32<C>(pages[o + v_off + tid + SA_CHUNK]);
         }
         __syncthreads();
     }
     const float inv = (l > 0.f ? 1.0f / l : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
-    A* o = out + ((size_t)t * H + h) * e;
-    if (tid < e) o[tid] = from_f32<A>(acc0 * inv);
-    if (tid + SA_CHUNK < e) o[tid + SA_CHUNK] = from_f32<A>(acc1 * inv);
+    O* o = out + ((size_t)t * H + h) * e;
+    if (tid < e) o[tid] = from_f32<O>(acc0 * inv);
+    if (tid + SA_CHUNK < e) o[tid + SA_CHUNK] = from_f32<O>(acc1 * inv);
 }
 
-extern "C" int aie_sink_attention_plain(const void* q, const void* pages, void* out, int dtype, const float* gate,
+extern "C" int aie_sink_attention_plain(const void* q, const void* pages, void* out, int dtype, int out_dtype, const float* gate,
                                         const float* temp, const float* slope, const float* sink, const int* positions,
                                         const int* token_req, const int* block_table, int bt_width, int num_pages,
                                         int P, int T, int H, int G, int d, int e, int window, int keep_first,
-                                        float scale, const int* token_list, unsigned* err, cudaStream_t stream) {
+                                        int chunk, int maps, float scale, const int* token_list, unsigned* err, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (d <= 0 || d > 2 * SA_CHUNK || e <= 0 || e > 2 * SA_CHUNK || G <= 0 || H % G || H > 65535) return AIE_UNSUPPORTED;
+    if (maps < 1 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     const size_t smem = (size_t)(((d + 1) & ~1) + SA_CHUNK + 32) * sizeof(float) + SA_CHUNK * sizeof(long long);
     dim3 grid(T, H);
-#define AIE_SA(A)                                                                                                      \
-    sink_attention_plain_kernel<A, A><<<grid, SA_CHUNK, smem, stream>>>(                                               \
-        (const A*)q, (const A*)pages, (A*)out, gate, temp, slope, sink, positions, token_req, block_table, bt_width,   \
-        num_pages, P, H, G, d, e, window, keep_first, scale, token_list, err)
-    if (dtype == AIE_F32) AIE_SA(float);
-    else if (dtype == AIE_BF16) AIE_SA(bf16);
+#define AIE_SA(A, O)                                                                                                   \
+    sink_attention_plain_kernel<A, A, O><<<grid, SA_CHUNK, smem, stream>>>(                                            \
+        (const A*)q, (const A*)pages, (O*)out, gate, temp, slope, sink, positions, token_req, block_table, bt_width,   \
+        num_pages, P, H, G, d, e, window, keep_first, chunk, maps, scale, token_list, err)
+    if (dtype == AIE_F32 && out_dtype == AIE_F32) AIE_SA(float, float);
+    else if (dtype == AIE_BF16 && out_dtype == AIE_BF16) AIE_SA(bf16, bf16);
+    else if (dtype == AIE_BF16 && out_dtype == AIE_F32) AIE_SA(bf16, float);
     else return AIE_BAD_ARG;
 #undef AIE_SA
     AIE_LAUNCH_CHECK();

@@ -6,6 +6,13 @@
 //   i reads j  iff  j <= i and (window <= 0 or i - j < window or j < keep_first)
 //   out_i = gate[i, h] * sum_j exp(s(i, j)) v_j / (exp(sink[h]) + sum_j exp(s(i, j)))
 //
+// chunk > 0 (without a window): i reads j  iff  j <= i and j / chunk == i / chunk.
+// maps > 1: a key/value head has `maps` keys in front of its one value, a row is [k_0 .. k_(maps-1) | v]; query head h
+// of the H (all maps counted) reads key h % maps of key/value head h / (H / G).  The prompt kernel's CTA loads the one
+// key its head reads; the decode kernel's CTA loads the whole row once for its heads of all maps (its DK is then all
+// keys of the row, and a head's query is zero outside its own map's elements).  Results are written in bfloat16, or
+// in float32 (out32) for a consumer that goes on in 32-bit.
+//
 // Scores, the running maximum and sum and the weights are float32.  A weight enters the product with the values
 // as two bfloat16 numbers (its rounded value and the rounded rest: 16 bits of mantissa), so that the tensor
 // cores add the same weights the float32 sum holds.
@@ -34,13 +41,13 @@ template <int D> __device__ __forceinline__ bf16* sk_at(bf16* base, int row, int
 }
 
 // One warp, 16 query rows against a tile of N keys in shared memory.  The thread holds rows (lane / 4) and
-// (lane / 4) + 8: their positions qp, factors qs (scale * temp) and slopes sl.  `masked`: apply the visibility
+// (lane / 4) + 8: their positions qp, the first keys low that they read, factors qs (scale * temp) and slopes sl.  `masked`: apply the visibility
 // rule (tiles wholly inside every row's sight skip it); keys above `key_end` are never visible.
 template <int DK, int DV, int N>
 __device__ __forceinline__ void sk_tile(const bf16* kb, const bf16* vb, const unsigned (&qf)[DK / 16][4],
                                         float (&o)[DV / 8][4], float (&m_run)[2], float (&l_run)[2], int kbase,
-                                        const int (&qp)[2], const float (&qs)[2], const float (&sl)[2], int window,
-                                        int keep_first, bool masked, int lane) {
+                                        const int (&qp)[2], const int (&low)[2], const float (&qs)[2],
+                                        const float (&sl)[2], int keep_first, bool masked, int lane) {
     float s[N / 8][4];
 #pragma unroll
     for (int j = 0; j < N / 8; ++j)
@@ -66,7 +73,7 @@ __device__ __forceinline__ void sk_tile(const bf16* kb, const bf16* vb, const un
             const int key = kbase + j * 8 + 2 * (lane & 3) + (e & 1);
             float v = s[j][e] * qs[i] - sl[i] * (float)(qp[i] - key);
             if (masked) {
-                const bool ok = key <= qp[i] && (window <= 0 || key > qp[i] - window || key < keep_first);
+                const bool ok = key <= qp[i] && (key >= low[i] || key < keep_first);
                 if (!ok) v = -INFINITY;
             }
             s[j][e] = v;
@@ -128,6 +135,12 @@ __device__ __forceinline__ void sk_tile(const bf16* kb, const bf16* vb, const un
     }
 }
 
+// first key that a query at `pos` reads (kept first keys aside)
+__device__ __forceinline__ int sk_low(int pos, int window, int chunk) {
+    if (chunk > 0) return pos / chunk * chunk;
+    return window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
+}
+
 template <int DK, int DV>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, bf16* __restrict__ out,
@@ -135,9 +148,10 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
                     const float* __restrict__ sink, const int* __restrict__ tiles, const int* __restrict__ q_start,
                     const int* __restrict__ q_len, const int* __restrict__ ctx_len,
                     const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G,
-                    int window, int keep_first, float scale, unsigned* err) {
-    constexpr int N = 64, W = DK + DV;
-    constexpr int CK = DK / 8, CV = DV / 8, CW = W / 8;      // 16-byte chunks of a key, a value, a cache row
+                    int window, int keep_first, int chunk, int maps, float scale, float* __restrict__ out32,
+                    unsigned* err) {
+    constexpr int N = 64;
+    constexpr int CK = DK / 8, CW = (DK + DV) / 8;           // 16-byte pieces of a key; of a key and a value
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);            // [128][DK]
     bf16* k_s = q_s + SK_M * DK;                               // [2][64][DK]
@@ -148,6 +162,8 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
     const int tile_i = (int)gridDim.y - 1 - (int)blockIdx.y;   // the list holds the tiles fewest keys first
     const int r = tiles[2 * tile_i], q_off = tiles[2 * tile_i + 1];
     const int h = blockIdx.x, g = h / (H / G);
+    const int W = maps * DK + DV;                              // elements of a cache row
+    const int k_off = (h % maps) * DK, v_off = (maps - 1) * DK;      // of this head's key; of the value behind c * 8 >= DK
     const int t0 = q_start[r] + q_off;
     const int rows_valid = min(SK_M, q_len[r] - q_off);
     const int p0 = ctx_len[r] + q_off;              // position of the tile's first query
@@ -161,8 +177,7 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
     }
     cp_async_commit();
 
-    int lo_min = 0;
-    if (window > 0 && p0 - window + 1 > 0) lo_min = p0 - window + 1;
+    const int lo_min = sk_low(p0, window, chunk), lo_last = sk_low(p_last, window, chunk);
     const int kt_lo = lo_min / N, kt_hi = p_last / N;
     // tiles of kept first keys that lie before the window's first tile
     const int n_kept = (window > 0 && keep_first > 0) ? min(kt_lo, (keep_first + N - 1) / N) : 0;
@@ -188,7 +203,7 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
             const int row = i / CW, c = i % CW;
             const int prow = row_s[buf * N + row];
             const bool ok = prow >= 0;
-            const bf16* src = pages + (size_t)(ok ? prow : 0) * W + c * 8;
+            const bf16* src = pages + (size_t)(ok ? prow : 0) * W + c * 8 + (c < CK ? k_off : v_off);
             if (c < CK) cp_async16(sk_at<DK>(kd, row, c), src, ok);
             else cp_async16(sk_at<DV>(vd, row, c - CK), src, ok);
         }
@@ -210,6 +225,9 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
     int qp[2];
     qp[0] = p0 + warp * 16 + (lane >> 2);
     qp[1] = qp[0] + 8;
+    int low[2];
+    low[0] = sk_low(qp[0], window, chunk);
+    low[1] = sk_low(qp[1], window, chunk);
     float qs[2], sl[2];
     qs[0] = qs[1] = scale * (temp ? temp[h] : 1.f);
     sl[0] = sl[1] = slope ? slope[h] : 0.f;
@@ -233,8 +251,8 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
         }
         const int kbase = kt * N;
         // the rule is applied on tiles that touch the diagonal or the low edge of some row's window
-        const bool masked = (kbase + N - 1 > p0) || (window > 0 && kbase < p_last - window + 1);
-        sk_tile<DK, DV, N>(k_s + buf * N * DK, v_s + buf * N * DV, qf, o, m_run, l_run, kbase, qp, qs, sl, window,
+        const bool masked = (kbase + N - 1 > p0) || kbase < lo_last;
+        sk_tile<DK, DV, N>(k_s + buf * N * DK, v_s + buf * N * DV, qf, o, m_run, l_run, kbase, qp, low, qs, sl,
                            keep_first, masked, lane);
         __syncthreads();     // everyone is done with this buffer before it is loaded again
     }
@@ -244,6 +262,13 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
         const int row = warp * 16 + (lane >> 2) + i * 8;
         if (row >= rows_valid) continue;
         const float inv = (l_run[i] > 0.f ? 1.0f / l_run[i] : 0.f) * (gate ? gate[(size_t)(t0 + row) * H + h] : 1.f);
+        if (out32) {
+            float* dst = out32 + ((size_t)(t0 + row) * H + h) * DV + 2 * (lane & 3);
+#pragma unroll
+            for (int j = 0; j < DV / 8; ++j)
+                *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[j][i * 2] * inv, o[j][i * 2 + 1] * inv);
+            continue;
+        }
         bf16* dst = out + ((size_t)(t0 + row) * H + h) * DV + 2 * (lane & 3);
 #pragma unroll
         for (int j = 0; j < DV / 8; ++j)
@@ -278,8 +303,8 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
                    const float* __restrict__ temp, const float* __restrict__ slope, const float* __restrict__ sink,
                    const int* __restrict__ dec_tokens, const int* __restrict__ positions,
                    const int* __restrict__ token_req, const int* __restrict__ block_table, int bt_width,
-                   int num_pages, int P, int H, int G, int GC, int window, int keep_first, float scale, int S,
-                   unsigned* err) {
+                   int num_pages, int P, int H, int G, int GC, int window, int keep_first, int chunk, int maps,
+                   float scale, int S, float* __restrict__ out32, unsigned* err) {
     constexpr int W = DK + DV, CW = W / 8, CK = DK / 8;
     constexpr int STILE = SdStage<W>::keys, KS = DK / 16;
     extern __shared__ __align__(128) unsigned char sd_smem[];
@@ -299,8 +324,7 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
     bf16* stage0 = reinterpret_cast<bf16*>(sd_smem + (size_t)warp * SD_NST * SdSmem<DK, DV>::stage_bytes);
     int* rows_w = reinterpret_cast<int*>(sd_smem + SdSmem<DK, DV>::rows_off) + warp * STILE;
 
-    int lo = 0;
-    if (window > 0 && pos - window + 1 > 0) lo = pos - window + 1;
+    const int lo = sk_low(pos, window, chunk);
     const int kept = min(keep_first, lo);
     const int nk = kept + pos + 1 - lo;
     const int tiles_total = (nk + STILE - 1) / STILE;
@@ -347,13 +371,14 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
     // q as the A operand: row = head; rows ng .. 15 are zero
     unsigned qa[KS][2];
     {
-        const bf16* qp = q + ((size_t)t * H + hbase + (qrow < ng ? qrow : 0)) * DK;
+        const int hh = hbase + (qrow < ng ? qrow : 0);
+        const int dm = DK / maps, k_off = (hh % maps) * dm;     // elements of a map's query; where its key lies in the row
+        const bf16* qp = q + (size_t)t * H * dm + (size_t)hh * dm - k_off;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
-            const unsigned a = *reinterpret_cast<const unsigned*>(qp + ks * 16 + qcol);
-            const unsigned b = *reinterpret_cast<const unsigned*>(qp + ks * 16 + 8 + qcol);
-            qa[ks][0] = qrow < ng ? a : 0u;
-            qa[ks][1] = qrow < ng ? b : 0u;
+            const bool on = qrow < ng && ks * 16 >= k_off && ks * 16 < k_off + dm;
+            qa[ks][0] = on ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + qcol) : 0u;
+            qa[ks][1] = on ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + 8 + qcol) : 0u;
         }
     }
     const int hq = hbase + (qrow < ng ? qrow : 0);
@@ -467,7 +492,9 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
         if (whole) {
             if (sink) L += __expf(sink[h] - M);      // the sink counts once, with no value
             const float inv = (L > 0.f ? 1.0f / L : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
-            out[((size_t)t * H + h) * DV + e] = __float2bfloat16_rn(A * inv);
+            const size_t at = ((size_t)t * H + h) * DV + e;
+            if (out32) out32[at] = A * inv;
+            else out[at] = __float2bfloat16_rn(A * inv);
         } else {
             const size_t pi = ((size_t)di * H + h) * S + s;
             part_o[pi * DV + e] = L > 0.f ? A / L : 0.f;
@@ -481,7 +508,7 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
 __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                  bf16* __restrict__ out, const float* __restrict__ gate,
                                  const float* __restrict__ sink, const int* __restrict__ dec_tokens, int H, int DV,
-                                 int S) {
+                                 int S, float* __restrict__ out32) {
     __shared__ float w_s[SD_MAX_SPLITS];
     __shared__ float wsum_s;
     const int di = blockIdx.x, h = blockIdx.y;
@@ -507,12 +534,14 @@ __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* 
         const float* src = part_o + base * DV + e;
         float A = 0.f;
         for (int s = 0; s < S; ++s) A += w_s[s] * src[(size_t)s * DV];
-        out[((size_t)t * H + h) * DV + e] = __float2bfloat16_rn(A * inv);
+        const size_t at = ((size_t)t * H + h) * DV + e;
+        if (out32) out32[at] = A * inv;
+        else out[at] = __float2bfloat16_rn(A * inv);
     }
 }
 
 #define SK_DISPATCH(DK_, DV_, CALL)                                                        \
-    if (d == DK_ && e == DV_) { CALL(DK_, DV_); }
+    if (d == DK_ && e == DV_) { CALL(DK_, DV_) }
 
 #define SK_DISPATCH_ALL(CALL)                                                              \
     SK_DISPATCH(32, 32, CALL) else SK_DISPATCH(32, 64, CALL) else SK_DISPATCH(32, 128, CALL) \
@@ -521,14 +550,16 @@ __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* 
     else return AIE_UNSUPPORTED;
 
 // Portions of prompts.  tiles: int32 [n, 2] = (request row, offset of a tile of 128 tokens among the tokens it
-// brings), fewest keys first.  q [T, H, d], out [T, H, e] bfloat16; pages [num_pages, G, P, d + e] bfloat16.
+// brings), fewest keys first.  q [T, H, d], out [T, H, e] bfloat16 (or out32 float32); pages [num_pages, G, P,
+// maps * d + e] bfloat16.
 extern "C" int aie_sink_attention_prefill(const void* q, const void* pages, void* out, const float* gate,
                                           const float* temp, const float* slope, const float* sink, const int* tiles,
                                           int n_tiles, const int* q_start, const int* q_len, const int* ctx_len,
                                           const int* block_table, int bt_width, int num_pages, int P, int H, int G,
-                                          int d, int e, int window, int keep_first, float scale, unsigned* err,
-                                          cudaStream_t stream) {
+                                          int d, int e, int window, int keep_first, int chunk, int maps, float scale,
+                                          float* out32, unsigned* err, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
+    if (maps < 1 || G <= 0 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     if (G <= 0 || H % G || n_tiles > 65535) return AIE_UNSUPPORTED;
     dim3 grid(H, n_tiles);
 #define SK_PRE(DK_, DV_)                                                                                              \
@@ -538,7 +569,8 @@ extern "C" int aie_sink_attention_prefill(const void* q, const void* pages, void
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
         kern<<<grid, SK_WARPS * 32, smem, stream>>>((const bf16*)q, (const bf16*)pages, (bf16*)out, gate, temp, slope, \
                                                     sink, tiles, q_start, q_len, ctx_len, block_table, bt_width,      \
-                                                    num_pages, P, H, G, window, keep_first, scale, err);              \
+                                                    num_pages, P, H, G, window, keep_first, chunk, maps, scale,       \
+                                                    out32, err);                                                      \
     }
     SK_DISPATCH_ALL(SK_PRE)
 #undef SK_PRE
@@ -551,9 +583,10 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
                                          const float* gate, const float* temp, const float* slope, const float* sink,
                                          const int* dec_tokens, int n, const int* positions, const int* token_req,
                                          const int* block_table, int bt_width, int num_pages, int P, int H, int G,
-                                         int d, int e, int window, int keep_first, float scale, int S, unsigned* err,
-                                         cudaStream_t stream) {
+                                         int d, int e, int window, int keep_first, int chunk, int maps, float scale,
+                                         int S, float* out32, unsigned* err, cudaStream_t stream) {
     if (n <= 0) return 0;
+    if (maps < 1 || G <= 0 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     if (G <= 0 || H % G || S < 1 || S > SD_MAX_SPLITS || n > 65535 || (S > 1 && (!part_o || !part_lse)))
         return AIE_UNSUPPORTED;
     const int group = H / G, GC = group < SD_HEADS ? group : SD_HEADS;
@@ -568,14 +601,16 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
         kern<<<grid, SD_WARPS * 32, smem, stream>>>((const bf16*)q, (const bf16*)pages, (bf16*)out, part_o, part_lse, \
                                                     gate, temp, slope, sink, dec_tokens, positions, token_req,        \
                                                     block_table, bt_width, num_pages, P, H, G, GC, window,            \
-                                                    keep_first, scale, S, err);                                       \
+                                                    keep_first, chunk, maps, scale, S, out32, err);                   \
     }
+    d *= maps;                       // the kernel's keys are all keys of a row
+    SK_DISPATCH(256, 32, SK_DEC) else SK_DISPATCH(256, 64, SK_DEC) else SK_DISPATCH(256, 128, SK_DEC) else
     SK_DISPATCH_ALL(SK_DEC)
 #undef SK_DEC
     if (S > 1) {
         const cudaError_t e1 = cudaGetLastError();
         if (e1 != cudaSuccess) return (int)e1;
-        sink_join_kernel<<<dim3(n, H), 128, 0, stream>>>(part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S);
+        sink_join_kernel<<<dim3(n, H), 128, 0, stream>>>(part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S, out32);
     }
     AIE_LAUNCH_CHECK();
 }

@@ -9,6 +9,7 @@ import os
 from ctypes import c_float, c_int, c_longlong, c_void_p
 from typing import Optional
 
+import numpy as np
 import torch
 
 from .loader import KernelError, check, library, require_cuda
@@ -67,8 +68,8 @@ def sm_count() -> int:
 
 # ---------------------------------------------------------------------------
 def embed_gather(ids: torch.Tensor, table: torch.Tensor, err: torch.Tensor,
-                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """x[t] = float32(table[ids[t]]); an id outside the table sets the error word."""
+                 out: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
+    """x[t] = float32(table[ids[t]]) * scale; an id outside the table sets the error word."""
     _dev(ids, table, err)
     T, (V, D) = ids.shape[0], table.shape
     if out is None:
@@ -76,7 +77,7 @@ def embed_gather(ids: torch.Tensor, table: torch.Tensor, err: torch.Tensor,
     lib = library("elementwise.cu")
     with region("embed_gather", T * D * table.element_size() + _nb(out)):
         check(lib.aie_embed_gather(_p(ids), _p(table), c_int(dtype_code(table)), _p(out), c_int(T),
-                                   c_int(D), c_int(V), _p(err), _stream()), "embed_gather")
+                                   c_int(D), c_int(V), c_float(scale), _p(err), _stream()), "embed_gather")
     return out
 
 
@@ -749,13 +750,14 @@ def expert_combine(y: torch.Tensor, pair_row: torch.Tensor, top: int, weight: fl
 
 def latent_prepare(proj: torch.Tensor, H: int, d: int, rot: int, rank: int, c_weight: Optional[torch.Tensor],
                    eps: float, inv_freq: torch.Tensor, pages: torch.Tensor, ctx, block_table: torch.Tensor,
-                   q_dtype: torch.dtype, write: bool, kv: Optional[torch.Tensor] = None, halves: bool = False):
+                   q_dtype: torch.dtype, write: bool, kv: Optional[torch.Tensor] = None, halves: bool = False,
+                   magnitude: float = 1.0):
     """From the fused projection [q heads (d plain | rot rotated) | latent (rank) | shared key part (rot)] of a
     step: (q_plain [T, H, d] in q_dtype, q_full [T, H, rank + rot] float32 whose last rot columns hold the
     rotated query parts); with `write`, the normalised latent and the rotated key part go into the tokens'
     cache rows.  pages [num_pages, 1, P, rank + rot].  kv: the latent and the key part come from this float32 view
     [T, >= rank + rot] (rows any stride) instead of the columns behind the queries.  halves: the rotation pairs
-    element i with i + rot_dims / 2 instead of 2i with 2i + 1."""
+    element i with i + rot_dims / 2 instead of 2i with 2i + 1.  magnitude: factor of all cosines and sines."""
     _dev(proj, c_weight, inv_freq, pages, block_table)
     T, ld = proj.shape
     need = H * (d + rot) + ((rank + rot) if write and kv is None else 0)
@@ -773,19 +775,22 @@ def latent_prepare(proj: torch.Tensor, H: int, d: int, rot: int, rank: int, c_we
                                      _p(pages), c_int(dtype_code(pages)), _p(ctx.positions), _p(ctx.token_req),
                                      _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[0]),
                                      c_int(pages.shape[2]), _p(ctx.err), _p(kv), c_int(kv.stride(0) if kv is not None else 0),
-                                     c_int(1 if halves else 0), _stream()), "latent_prepare")
+                                     c_int(1 if halves else 0), c_float(magnitude), _stream()), "latent_prepare")
     return q_plain, q_full
 
 
 def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table: torch.Tensor, rank: int,
-                     scale: float, window: int, out_dtype: torch.dtype, work=None) -> torch.Tensor:
+                     scale: float, window: int, out_dtype: torch.dtype, work=None,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """softmax over the visible cache rows of (q_full . row) * scale, times the rows' first `rank` elements:
     [T, H, rank].  q_full [T, H, dk] float32; pages [num_pages, 1, P, dk].  `work`: the step's units of tokens
     (`tiles` [n, 2], `tq`) for the tensor-core kernel, which bfloat16 takes when the sizes fit (a latent of
-    64 .. 512 in steps of 64, rows a multiple of 16); everything else takes the plain kernel."""
-    _dev(q_full, pages, block_table)
+    64 .. 512 in steps of 64, rows a multiple of 16); everything else takes the plain kernel.  sink [H] float32: the
+    denominator also holds exp(sink[h])."""
+    _dev(q_full, pages, block_table, sink)
     T, H, dk = q_full.shape
-    if q_full.dtype != torch.float32 or pages.shape[3] != dk or pages.shape[1] != 1:
+    if (q_full.dtype != torch.float32 or pages.shape[3] != dk or pages.shape[1] != 1
+            or (sink is not None and (sink.dtype != torch.float32 or sink.shape != (H,)))):
         raise KernelError("latent_attention: shapes or dtypes do not fit")
     out = torch.empty((T, H, rank), dtype=out_dtype, device=q_full.device)
     cost = (float(_nb(q_full, out)), 0.0)
@@ -816,7 +821,7 @@ def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table
                                               _p(ctx.q_len), _p(ctx.ctx_len), _p(block_table), c_int(block_table.shape[1]),
                                               c_int(pages.shape[0]), c_int(pages.shape[2]), c_int(T), c_int(H),
                                               c_int(rank), c_int(dk), c_int(window), c_float(scale), c_int(splits),
-                                              _p(ctx.err), _stream()), "latent_attention_tc")
+                                              _p(sink), _p(ctx.err), _stream()), "latent_attention_tc")
         return out
     lib = library("latent_attention.cu")
     with region("latent_attention", *cost):
@@ -824,7 +829,7 @@ def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table
                                        c_int(dtype_code(out)), _p(ctx.positions), _p(ctx.token_req), _p(block_table),
                                        c_int(block_table.shape[1]), c_int(pages.shape[0]), c_int(pages.shape[2]),
                                        c_int(T), c_int(H), c_int(rank), c_int(dk), c_int(window), c_float(scale),
-                                       _p(ctx.err), _stream()), "latent_attention")
+                                       _p(sink), _p(ctx.err), _stream()), "latent_attention")
     return out
 
 
@@ -1133,23 +1138,30 @@ def sink_attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], pages: t
 
 
 SINK_FAST_SIZES = (32, 64, 128)      # key and value sizes of the tensor-core kernels of sink_attention
+SINK_FAST_ROWS = (32, 64, 128, 256)  # all keys of a cache row (maps * key size) that the split-KV kernel takes
 
 
 def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Tensor], temp: Optional[torch.Tensor],
                    slope: Optional[torch.Tensor], sink: Optional[torch.Tensor], ctx, work, block_table: torch.Tensor,
-                   e: int, scale: float, window: int, keep_first: int) -> torch.Tensor:
+                   e: int, scale: float, window: int, keep_first: int, chunk: int = 0, maps: int = 1,
+                   out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """Attention of a step's query tokens over cache rows [k (d) | v (e)]:
     s(i, j) = (q_i . k_j) * scale * temp[h] - slope[h] * (i - j) over the keys j <= i with i - j < window or
     j < keep_first (window 0: all); softmax whose denominator also holds exp(sink[h]); times gate[i, h].
-    q [T, H, d]; gate [T, H], temp, slope, sink [H] float32 or None.  Returns [T, H, e] in q's dtype.
+    q [T, H, d]; gate [T, H], temp, slope, sink [H] float32 or None.  Returns [T, H, e] in q's dtype or `out_dtype`
+    (float32).  chunk > 0 (without a window): a query reads the keys of its own chunk of that many positions only.
+    maps > 1: rows are [k_0 .. k_(maps-1) | v] and query head h (H counts the heads of all maps) reads key h % maps.
     bfloat16 with key and value sizes of 32, 64 or 128: lone tokens take the split-KV kernel, portions of prompts
     the tiled tensor-core kernel (`work`: the attention work lists); everything else takes the plain kernel."""
     _dev(q, pages, gate, temp, slope, sink, block_table)
     T, H, d = q.shape
     G = pages.shape[1]
-    if pages.shape[3] != d + e or H % G or pages.dtype != q.dtype:
-        raise KernelError("sink_attention: shapes or dtypes do not fit")
-    out = torch.empty((T, H, e), dtype=q.dtype, device=q.device)
+    out_dtype = out_dtype or q.dtype
+    if (pages.shape[3] != maps * d + e or H % (G * maps) or pages.dtype != q.dtype or out_dtype not in (q.dtype, torch.float32)
+            or (chunk and (window or keep_first))):
+        raise KernelError("sink_attention: shapes, dtypes or masks do not fit")
+    out = torch.empty((T, H, e), dtype=out_dtype, device=q.device)
+    out32 = out if out_dtype == torch.float32 else None
     cost = (0.0, 0.0)
     if _profiling() and hasattr(ctx, "h_q_len"):
         ql, cl = ctx.h_q_len.astype(float), ctx.h_ctx_len.astype(float)
@@ -1157,15 +1169,21 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
         if window > 0:
             seen = seen.clip(max=float(window + keep_first))
         rows = (cl + ql).clip(max=float(window + keep_first) + ql) if window > 0 else cl + ql
-        cost = (float(rows.sum()) * G * (d + e) * pages.element_size() + _nb(q, out),
+        if chunk > 0:
+            pairs = [sum(p % chunk + 1 for p in range(int(c), int(c + n))) for n, c in zip(ql, cl)]
+            seen, rows = np.asarray(pairs, dtype=float) / ql, cl + ql - cl // chunk * chunk
+        cost = (float(rows.sum()) * G * (maps * d + e) * pages.element_size() + _nb(q, out),
                 2.0 * float((ql * seen).sum()) * H * (d + e))
-    if q.dtype == torch.bfloat16 and d in SINK_FAST_SIZES and e in SINK_FAST_SIZES:
+    if q.dtype == torch.bfloat16 and d in SINK_FAST_SIZES and e in SINK_FAST_SIZES and maps * d in SINK_FAST_ROWS:
         fast = library("sink_attention_tc.cu")
         common = (_p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[0]), c_int(pages.shape[2]),
-                  c_int(H), c_int(G), c_int(d), c_int(e), c_int(window), c_int(keep_first), c_float(scale))
+                  c_int(H), c_int(G), c_int(d), c_int(e), c_int(window), c_int(keep_first), c_int(chunk), c_int(maps),
+                  c_float(scale))
         if work.n_decode:
             n = work.n_decode
             keys = work.max_decode_len if window <= 0 else min(window + keep_first, work.max_decode_len)
+            if chunk > 0:
+                keys = min(keys, chunk)
             S = min(decode_splits(n, G, H // G, keys), 64)
             part_o = part_lse = None
             if S > 1:
@@ -1176,23 +1194,24 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
                 check(fast.aie_sink_attention_decode(_p(q), _p(pages), _p(out), _p(part_o), _p(part_lse), _p(gate),
                                                      _p(temp), _p(slope), _p(sink), _p(work.decode_tokens), c_int(n),
                                                      _p(ctx.positions), _p(ctx.token_req), *common, c_int(S),
-                                                     _p(ctx.err), _stream()), "sink_attention_decode")
+                                                     _p(out32), _p(ctx.err), _stream()), "sink_attention_decode")
         if work.n_decode < ctx.R:
             tiles = work.prefill_tiles
             share = 1.0 - float(work.n_decode) / T
             with region("sink_attention_prefill", cost[0] * share, cost[1] * share):
                 check(fast.aie_sink_attention_prefill(_p(q), _p(pages), _p(out), _p(gate), _p(temp), _p(slope), _p(sink),
                                                       _p(tiles), c_int(tiles.shape[0]), _p(ctx.q_start), _p(ctx.q_len),
-                                                      _p(ctx.ctx_len), *common, _p(ctx.err), _stream()),
+                                                      _p(ctx.ctx_len), *common, _p(out32), _p(ctx.err), _stream()),
                       "sink_attention_prefill")
         return out
     lib = library("sink_attention.cu")
     with region("sink_attention_plain", *cost):
-        check(lib.aie_sink_attention_plain(_p(q), _p(pages), _p(out), c_int(dtype_code(q)), _p(gate), _p(temp), _p(slope),
-                                           _p(sink), _p(ctx.positions), _p(ctx.token_req), _p(block_table),
+        check(lib.aie_sink_attention_plain(_p(q), _p(pages), _p(out), c_int(dtype_code(q)), c_int(dtype_code(out)), _p(gate),
+                                           _p(temp), _p(slope), _p(sink), _p(ctx.positions), _p(ctx.token_req), _p(block_table),
                                            c_int(block_table.shape[1]), c_int(pages.shape[0]), c_int(pages.shape[2]),
                                            c_int(T), c_int(H), c_int(G), c_int(d), c_int(e), c_int(window),
-                                           c_int(keep_first), c_float(scale), _p(None), _p(ctx.err), _stream()),
+                                           c_int(keep_first), c_int(chunk), c_int(maps), c_float(scale), _p(None),
+                                           _p(ctx.err), _stream()),
               "sink_attention_plain")
     return out
 
@@ -1345,32 +1364,35 @@ def normed_attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_weig
                         k_weight: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rot_dims: int,
                         halves: bool, pages: torch.Tensor, ctx, block_table: torch.Tensor, H: int, G: int, d: int, e: int,
                         mix_from: Optional[torch.Tensor] = None, mix_lambda: Optional[torch.Tensor] = None,
-                        keep_values: bool = False, write: bool = True):
+                        keep_values: bool = False, write: bool = True, maps: int = 1, per_head: bool = False):
     """From a step's fused projection whose first columns are [q (H d) | k (G d) | v (G e)] (float32 [T, >= that]):
     biases added; all of q divided by its root mean square over the H d elements, times q_weight (k likewise; None: no
     norm); the first rot_dims elements of every head of q and k rotated by the token's position (pairs of neighbours,
     or halves); v <- (1 - lambda) v + lambda mix_from[t] when mix_from [T, G e] float32 is given (lambda one float on
     the device).  q [T, H, d] in the cache's dtype is returned; with `write`, the token's cache row [k | v] is
     written.  keep_values: the values as they are cached are also returned in float32 [T, G e].
-    pages [num_pages, G, P, d + e]."""
+    pages [num_pages, G, P, d + e].  per_head: every head of q and of k is normed by itself, with weights [d].
+    maps > 1: k has G * maps heads, a row is [k_0 .. k_(maps-1) | v], and H counts the query heads of all maps."""
     _dev(proj, bias, q_weight, k_weight, inv_freq, pages, block_table, mix_from, mix_lambda)
     T, ld = proj.shape
-    n = H * d + G * (d + e)
-    if (proj.dtype != torch.float32 or ld < n or pages.shape[1] != G or pages.shape[3] != d + e
+    n = H * d + G * (maps * d + e)
+    nq, nk = (d, d) if per_head else (H * d, G * maps * d)
+    if (proj.dtype != torch.float32 or ld < n or pages.shape[1] != G or pages.shape[3] != maps * d + e
             or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != n))
-            or (q_weight is not None and (k_weight is None or q_weight.numel() != H * d or k_weight.numel() != G * d))
+            or (q_weight is not None and (k_weight is None or q_weight.numel() != nq or k_weight.numel() != nk))
             or (mix_from is not None and (mix_from.dtype != torch.float32 or mix_from.shape != (T, G * e) or mix_lambda is None))):
         raise KernelError("normed_attn_prepare: shapes or dtypes do not fit")
     q = torch.empty((T, H, d), dtype=pages.dtype, device=proj.device)
     kept = torch.empty((T, G * e), dtype=torch.float32, device=proj.device) if keep_values else None
     lib = library("sink_attention.cu")
-    with region("normed_attn_prepare", T * n * 4 + _nb(q, kept, mix_from) + T * G * (d + e) * pages.element_size()):
+    with region("normed_attn_prepare", T * n * 4 + _nb(q, kept, mix_from) + T * G * (maps * d + e) * pages.element_size()):
         check(lib.aie_normed_attn_prepare(_p(proj), c_int(ld), _p(bias), _p(q_weight), _p(k_weight), c_float(eps),
                                           _p(inv_freq), c_int(rot_dims), c_int(1 if halves else 0), _p(mix_from),
                                           _p(mix_lambda), _p(kept), _p(q), _p(pages), c_int(dtype_code(pages)),
                                           _p(ctx.positions), _p(ctx.token_req), _p(block_table), c_int(block_table.shape[1]),
                                           c_int(pages.shape[0]), c_int(pages.shape[2]), c_int(T), c_int(H), c_int(G), c_int(d),
-                                          c_int(e), c_int(1 if write else 0), _p(ctx.err), _stream()), "normed_attn_prepare")
+                                          c_int(e), c_int(maps), c_int(1 if per_head else 0), c_int(1 if write else 0),
+                                          _p(ctx.err), _stream()), "normed_attn_prepare")
     return q, kept
 
 
@@ -1387,3 +1409,144 @@ def slice_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: 
         check(lib.aie_slice_rmsnorm(_p(x), c_int(x.stride(0)), _p(weight), _p(out), c_int(dtype_code(out)), c_int(T), c_int(n),
                                     c_float(eps), _stream()), "slice_rmsnorm")
     return out
+
+
+# ---------------------------------------------------------------------------
+# parts of layers that gate and norm a sublayer's result before it joins the stream, shift their mixer's input towards
+# the token before, take a learned input per token, and mix with two attention maps
+class ExpertRows:
+    """What a mixture of experts leaves for its consumer to sum: rows `y` [rows, D] float32 of (token, choice) pairs,
+    `pair_row` [T * top] (a pair's row) and `weights` [T, top] float32."""
+
+    def __init__(self, y: torch.Tensor, pair_row: torch.Tensor, weights: torch.Tensor):
+        self.y, self.pair_row, self.weights = y, pair_row, weights
+
+
+def token_shift(x: torch.Tensor, shift: torch.Tensor, state: torch.Tensor, ctx, out_dtype: torch.dtype,
+                plain: bool = False):
+    """x + (x' - x) * shift with x' the row of the request's token before (its state [max_seqs, D] for the first token
+    of a step; the state becomes the last row).  x [T, D], shift [D], state float32.  plain: also returns x itself in
+    out_dtype (x where that is float32): (shifted, x)."""
+    _dev(x, shift, state)
+    T, D = x.shape
+    if any(t.dtype != torch.float32 for t in (x, shift, state)) or shift.shape != (D,) or state.shape[1:] != (D,):
+        raise KernelError("token_shift: a float32 stream [T, D], weights [D] and state [slots, D]")
+    out = torch.empty((T, D), dtype=out_dtype, device=x.device)
+    same = torch.empty((T, D), dtype=out_dtype, device=x.device) if plain and out_dtype != x.dtype else None
+    lib = library("gated_stream.cu")
+    with region("token_shift", _nb(x, out, same)):
+        check(lib.aie_token_shift(_p(x), _p(shift), _p(state), _p(out), _p(same), c_int(dtype_code(out)), _p(ctx.q_start),
+                                  _p(ctx.q_len), _p(ctx.slots), _p(ctx.token_req), c_int(T), c_int(D),
+                                  c_int(state.shape[0]), _p(ctx.err), _stream()), "token_shift")
+    return (out, same if same is not None else x) if plain else out
+
+
+def gated_norm_add(x: torch.Tensor, y, weight: torch.Tensor, eps: float, out_dtype: Optional[torch.dtype] = None,
+                   gate: Optional[torch.Tensor] = None, gate_bias: Optional[torch.Tensor] = None,
+                   bias: Optional[torch.Tensor] = None, next_shift=None, ctx=None):
+    """x += norm((y + bias) * sigmoid(gate + gate_bias)) * weight in place, norm(u) = u / sqrt(mean(u^2) + eps), all in
+    float32.  y: float32 [T, D], [parts, T, D] (parts of a split product), or ExpertRows (summed here by weight).  gate:
+    logits float32, the first D columns of a view [T, >= D] or [parts, T, >= D] with any row stride.  out_dtype: also returns the new x in
+    that dtype (x itself where that is float32).  next_shift = (shift [D], state [slots, D]), for steps in which every
+    request brings one token: returns (new x, token_shift of it) in out_dtype and replaces the state."""
+    _dev(x, weight, gate_bias, bias)
+    T, D = x.shape
+    f32 = torch.float32
+    if x.dtype != f32 or weight.dtype != f32 or weight.shape != (D,) or any(
+            t is not None and (t.dtype != f32 or t.shape != (D,)) for t in (gate_bias, bias)):
+        raise KernelError("gated_norm_add: stream, weight and biases are float32, one number per column")
+    pair_row = weights = None
+    top = parts = stride = 0
+    if isinstance(y, ExpertRows):
+        rows, pair_row, weights = y.y, y.pair_row, y.weights
+        _dev(rows, pair_row, weights)
+        top = weights.shape[1]
+        if rows.dtype != f32 or rows.shape[1] != D or weights.dtype != f32 or weights.shape[0] != T or pair_row.numel() != T * top \
+                or bias is not None:
+            raise KernelError("gated_norm_add: expert rows do not fit")
+        nb = T * top * D * 4
+    else:
+        rows = y
+        _dev(rows)
+        if rows.dtype != f32 or rows.shape[-2:] != (T, D):
+            raise KernelError("gated_norm_add: a branch is float32 [T, D] or [parts, T, D]")
+        parts, stride = (rows.shape[0], rows.stride(0)) if rows.dim() == 3 else (1, 0)
+        nb = _nb(rows)
+    zparts, zstride, ldz = 0, 0, 0
+    if gate is not None:
+        if gate.dtype != f32 or gate.shape[-2] != T or gate.shape[-1] < D or gate.stride(-1) != 1:
+            raise KernelError("gated_norm_add: gate logits are float32 [(parts,) T, >= D]")
+        zparts, zstride = (gate.shape[0], gate.stride(0)) if gate.dim() == 3 else (1, 0)
+        ldz = gate.stride(-2)
+        nb += zparts * T * D * 4
+    code = dtype_code(out_dtype or f32)
+    out = torch.empty((T, D), dtype=out_dtype, device=x.device) if out_dtype is not None and out_dtype != f32 else None
+    shift = state = shifted = None
+    if next_shift is not None:
+        shift, state = next_shift
+        _dev(shift, state)
+        if ctx is None or ctx.max_q_len != 1 or state.shape[1:] != (D,) or shift.shape != (D,) or out_dtype is None:
+            raise KernelError("gated_norm_add: the next layer's shift is made in steps of lone tokens only")
+        shifted = torch.empty((T, D), dtype=out_dtype, device=x.device)
+        nb += 2 * T * D * 4
+    lib = library("gated_stream.cu")
+    with region("gated_norm_add", 2 * _nb(x) + nb + _nb(out, shifted)):
+        check(lib.aie_gated_norm_add(
+            _p(x), _p(rows), c_int(parts), c_longlong(stride), _p(bias), _p(pair_row), _p(weights), c_int(top), _p(gate),
+            c_int(zparts), c_longlong(zstride), c_int(ldz), _p(gate_bias), _p(weight), _p(out), c_int(code), c_int(T),
+            c_int(D), c_float(eps), _p(shift), _p(state), _p(shifted), _p(ctx.slots if ctx is not None else None),
+            _p(ctx.token_req if ctx is not None else None), c_int(state.shape[0] if state is not None else 0),
+            _p(ctx.err if ctx is not None else None), _stream()), "gated_norm_add")
+    new = out if out is not None else x
+    return (new, shifted) if next_shift is not None else new
+
+
+def side_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, offset: int, n: int, out_dtype: torch.dtype,
+              err: torch.Tensor) -> torch.Tensor:
+    """gelu_tanh(z[t, c]) * table[ids[t], offset + c] for c < n, in float32.  z float32 [T, >= n] or [parts, T, >= n]
+    (parts of a split product, added first)."""
+    _dev(ids, table, err)
+    if z.dtype != torch.float32 or z.shape[-1] < n or z.stride(-1) != 1 or offset + n > table.shape[1]:
+        raise KernelError("side_gate: shapes or dtypes do not fit")
+    T = z.shape[-2]
+    parts, stride = (z.shape[0], z.stride(0)) if z.dim() == 3 else (1, 0)
+    out = torch.empty((T, n), dtype=out_dtype, device=z.device)
+    lib = library("gated_stream.cu")
+    with region("side_gate", parts * T * n * 4 + T * n * table.element_size() + _nb(out)):
+        check(lib.aie_side_gate(_p(z), c_int(parts), c_longlong(stride), c_int(z.stride(-2)), _p(ids), _p(table),
+                                c_int(dtype_code(table)), c_int(table.shape[0]), c_int(table.shape[1]), c_int(offset),
+                                _p(out), c_int(dtype_code(out)), c_int(T), c_int(n), _p(err), _stream()), "side_gate")
+    return out
+
+
+def map_difference(a: torch.Tensor, lam: float, eps: float, factor: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """a [T, 2 H, e] float32, a head's two maps side by side: o = a_1 - lam a_2, out = o / sqrt(mean(o^2) + eps) * factor
+    over the head's e values; [T, H * e]."""
+    _dev(a)
+    T, H2, e = a.shape
+    if a.dtype != torch.float32 or H2 % 2:
+        raise KernelError("map_difference: float32 [T, 2 H, e]")
+    out = torch.empty((T, H2 // 2 * e), dtype=out_dtype, device=a.device)
+    lib = library("gated_stream.cu")
+    with region("map_difference", _nb(a, out)):
+        check(lib.aie_map_difference(_p(a), c_float(lam), c_float(eps), c_float(factor), _p(out), c_int(dtype_code(out)),
+                                     c_longlong(T * (H2 // 2)), c_int(e), _stream()), "map_difference")
+    return out
+
+
+def route_chosen(z: torch.Tensor, bias: Optional[torch.Tensor], E: int, top: int):
+    """(ids int32 [T, top], weights float32 [T, top]): the `top` largest of the logits z + bias per token and the softmax
+    over those.  z float32 [T, >= E] or [parts, T, >= E] with any row stride, bias [E] float32 or None."""
+    _dev(bias)
+    if z.dtype != torch.float32 or z.shape[-1] < E or z.stride(-1) != 1 or (bias is not None and (
+            bias.dtype != torch.float32 or bias.shape != (E,))):
+        raise KernelError("route_chosen: float32 logits and bias")
+    T = z.shape[-2]
+    parts, stride = (z.shape[0], z.stride(0)) if z.dim() == 3 else (1, 0)
+    ids = torch.empty((T, top), dtype=torch.int32, device=z.device)
+    weights = torch.empty((T, top), dtype=torch.float32, device=z.device)
+    lib = library("gated_stream.cu")
+    with region("route_chosen", parts * T * E * 4 + _nb(ids, weights)):
+        check(lib.aie_route_chosen(_p(z), c_int(parts), c_longlong(stride), c_int(z.stride(-2)), _p(bias), c_int(T), c_int(E),
+                                   c_int(top), _p(ids), _p(weights), _stream()), "route_chosen")
+    return ids, weights

@@ -1,12 +1,13 @@
 from .attention import ATTENTION_WORK, AttentionWork, GQAAttention
 from .base import (Block, BuildEnv, CacheNeed, FeedForward, KVRequest, LayerCache, Mixer, Norm, Part,
                    PositionEncoding, StateRequest, StepPlanner, TokenFilter)
-from .block import DepthAveragedBlock, ParallelBlock, PreNormBlock, SandwichNormBlock
+from .block import DepthAveragedBlock, GatedPostNormBlock, ParallelBlock, PreNormBlock, SandwichNormBlock
 from .conv import CausalShortConv
 from .embedding import LMHead, TokenEmbedding
 from .latent_attention import LATENT_WORK, LatentAttention, LatentWork
 from .linear_attention import DecayLinearAttention, ForgetGateLinearAttention
 from .delta_rule import GatedDeltaRule
+from .differential_attention import DifferentialAttention
 from .mlp import DenseFF, PolyNormFF, SwiGLU
 from .moe import RoutedMoE, TableMoE
 from .parallel import ParallelMixers
@@ -18,8 +19,10 @@ from .norm import DynamicTanh, RMSNorm
 from .normed_attention import NormedGatedAttention
 from .registry import (lookup, register, register_block, register_feed_forward, register_mixer,
                        register_norm, register_position_encoding)
-from .rope import RotaryEncoding, rotary_inv_freq
+from .rope import RotaryEncoding, rotary_inv_freq, rotary_magnitude
 from .spec import LayerSpec, ModelSpec, PartSpec, RunStep
+from .token_shift import TokenShift
+from .token_side import TokenSide
 
 register("mixer", "gqa_attention", GQAAttention)
 register("feed_forward", "swiglu", SwiGLU)
@@ -46,6 +49,10 @@ register("norm", "dynamic_tanh", DynamicTanh)
 register("block", "parallel_depth_average", ParallelBlock)
 register("mixer", "forget_gate_linear_attention", ForgetGateLinearAttention)
 register("mixer", "normed_gated_attention", NormedGatedAttention)
+register("mixer", "differential_attention", DifferentialAttention)
+register("filter", "token_shift", TokenShift)
+register("feed_forward", "token_side", TokenSide)
+register("block", "gated_post_norm", GatedPostNormBlock)
 
 __all__ = ["ATTENTION_WORK", "AttentionWork", "GQAAttention", "Block", "BuildEnv", "CacheNeed", "FeedForward",
            "KVRequest", "LayerCache", "Mixer", "Norm", "Part", "PositionEncoding", "StateRequest", "StepPlanner", "PreNormBlock", "LMHead",
@@ -55,4 +62,5 @@ __all__ = ["ATTENTION_WORK", "AttentionWork", "GQAAttention", "Block", "BuildEnv
            "LayerSpec", "ModelSpec", "PartSpec", "RunStep", "TokenFilter", "DepthAveragedBlock", "CausalShortConv",
            "LatentAttention", "DecayLinearAttention", "PolyNormFF", "TableMoE", "SandwichNormBlock", "ParallelMixers",
            "ScalarDecayStateSpace", "RoutedMoE", "SinkWindowAttention", "GatedDeltaRule", "DenseFF", "SinusoidalPositions",
-           "DynamicTanh", "ParallelBlock", "ForgetGateLinearAttention", "NormedGatedAttention"]
+           "DynamicTanh", "ParallelBlock", "ForgetGateLinearAttention", "NormedGatedAttention", "DifferentialAttention", "TokenShift", "TokenSide",
+           "GatedPostNormBlock", "rotary_magnitude"]

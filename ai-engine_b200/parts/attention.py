@@ -74,6 +74,8 @@ class GQAAttention(Mixer):
         rot = self.rope.rotation() if self.rope is not None else None
         if self.rope is not None and getattr(self.rope, "interleaved", False):
             raise ValueError("attention: its kernels rotate split halves; an interleaved encoding is not taken")
+        if self.rope is not None and getattr(self.rope, "magnitude", 1.0) != 1.0:
+            raise ValueError("attention: its kernels rotate without a magnitude; a yarn encoding is not taken")
         if rot is not None and rot[1] > self.d:
             raise ValueError("attention: rotary width exceeds head_dim")
         self.taps = int(p.get("qk_conv") or 0)

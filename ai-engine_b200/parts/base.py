@@ -34,6 +34,7 @@ class KVRequest:
     planes: int = 2      # 2: keys and values; 1: one vector per token and kv head (a compressed cache, or a key and
     #                      a value of another size side by side in one row)
     keep_first: int = 0  # with a window: the first `keep_first` keys stay readable for every later query
+    chunk: int = 0       # > 0: a query at p reads the keys of its own chunk only, from p // chunk * chunk on
 
 
 @dataclass(frozen=True)
@@ -154,6 +155,9 @@ class Mixer(Part):
     # True: forward takes `add_to=stream` (the float32 residual stream) and may add its output there itself,
     # returning None instead of the output (a block then hands no pending branch to the next norm)
     adds_in_place = False
+    # True: the output projection has a bias, kept as `output_bias` (float32 [hidden]); forward takes `leave_bias=True`,
+    # with which the caller adds it itself
+    leaves_bias = False
 
     def forward(self, h: torch.Tensor, ctx, cache: LayerCache) -> torch.Tensor:
         raise NotImplementedError
@@ -163,6 +167,10 @@ class FeedForward(Part):
     """Token-local: forward(h [T, hidden], ctx) -> [T, hidden], float32 or the compute dtype."""
 
     adds_in_place = False      # as for a Mixer
+    # True: forward takes `leave_rows=True`, with which it returns ops.ExpertRows (a token's expert rows and their
+    # weights) for a caller that sums them itself, and `logits=` (float32 [(parts,) T, n]) for the product of its
+    # input with the weight that `router_weight()` hands out, when the caller has made it along with one of its own
+    leaves_rows = False
 
     def forward(self, h: torch.Tensor, ctx) -> torch.Tensor:
         raise NotImplementedError

@@ -230,3 +230,110 @@ class ParallelBlock(Block):
         if made is not None:
             ctx.normed_ahead = (nxt, made)
         return x, None
+
+
+class GatedPostNormBlock(Block):
+    """A block whose sublayers read the stream as it is and whose results are gated and normed before they join it:
+
+        y = mixer(shift(x)) * sigmoid(W_g1 x + b_g1);   x = x + mixer_norm(y)
+        y = ffn(x) * sigmoid(W_g2 x + b_g2);            x = x + ffn_norm(y)
+        x = x + side_norm(side(x))
+
+    Roles: `shift` (a filter over time in front of the mixer) is optional, so are the feed-forward with its norm, and
+    `side` (a token-local part that closes the layer) with its norm.  tensors: mixer_gate [hidden, hidden] with
+    mixer_gate_bias [hidden], ffn_gate with ffn_gate_bias (each pair optional: no gate).
+
+    The stream changes in one kernel a sublayer, which joins the parts of the products (or the expert rows), adds the
+    projection's bias, gates, norms, adds, and hands on the new stream in the compute dtype.  A router whose weight the
+    feed-forward hands out is a product with the feed-forward's gate.  In steps in which every request brings one
+    token the layer's last kernel makes the next layer's shift too (`set_next_block`) and hangs it on the step."""
+
+    roles = {"shift": "filter", "mixer": "mixer", "mixer_norm": "norm", "ffn": "feed_forward", "ffn_norm": "norm",
+             "side": "feed_forward", "side_norm": "norm"}
+    optional_roles = ("shift", "ffn", "ffn_norm", "side", "side_norm")
+
+    def __init__(self, spec, env, parts):
+        super().__init__(spec, env)
+        self.p = parts
+        self.hidden = env.hidden_size
+        if ("ffn" in parts) != ("ffn_norm" in parts) or ("side" in parts) != ("side_norm" in parts):
+            raise ValueError("post-norm block: a feed-forward and a side input come with their norms")
+        self.gated = [n for n in ("mixer_gate", "ffn_gate") if n in spec.tensors]
+        if "ffn_gate" in self.gated and "ffn" not in parts:
+            raise ValueError("post-norm block: a gate without a feed-forward")
+        self.gate, self.gate_bias = {}, {}
+        self.joined = False            # the feed-forward's gate and its router are one weight
+        self.next_block = None
+
+    def tensor_specs(self):
+        t = self.spec.tensors
+        return [s for n in self.gated for s in (TensorSpec(t[n], (self.hidden, self.hidden)),
+                                                TensorSpec(t[n + "_bias"], (self.hidden,), std=0.3))]
+
+    def load(self, source):
+        t = self.spec.tensors
+        for n in self.gated:
+            self.gate[n] = source.get(t[n])
+            self.gate_bias[n] = source.get(t[n + "_bias"]).float().contiguous()
+        ffn = self.p.get("ffn")
+        if ffn is not None and getattr(ffn, "leaves_rows", False) and "ffn_gate" in self.gate:
+            router = ffn.router_weight()
+            if router.dtype == self.gate["ffn_gate"].dtype:
+                self.gate["ffn_gate"] = torch.cat([self.gate["ffn_gate"], router], dim=0).contiguous()
+                self.joined = True
+
+    def weight_bytes(self):
+        return sum(w.numel() * w.element_size() for w in self.gate.values())
+
+    def flops(self, tokens, keys=0.0):
+        return 2.0 * tokens * self.hidden * self.hidden * len(self.gated)
+
+    def set_next_block(self, block) -> None:
+        """The block that runs after this one in every step (only when every layer runs once)."""
+        self.next_block = block if isinstance(block, GatedPostNormBlock) and hasattr(block.p.get("shift"), "ahead") else None
+
+    def forward(self, x, pending, ctx, caches):
+        if pending is not None:
+            raise RuntimeError("post-norm block: the block before it left a branch that no norm adds")
+        p, dt = self.p, self.env.dtype
+        ahead = getattr(ctx, "shifted_ahead", None)
+        if ahead is not None and ahead[0] is self:
+            h, shifted = ahead[1], ahead[2]
+        elif "shift" in p:
+            shifted, h = p["shift"].forward(x, ctx, caches["shift"], plain=True)
+        else:
+            h = shifted = ops.cast(x, dt)
+        ctx.shifted_ahead = None
+        z = ops.linear_parts(h, self.gate["mixer_gate"], ctx.err) if "mixer_gate" in self.gate else None
+        mixer = p["mixer"]
+        y = mixer.forward(shifted, ctx, caches.get("mixer"), **(dict(leave_bias=True) if mixer.leaves_bias else {}))
+        bias = mixer.output_bias if mixer.leaves_bias else None
+        last = "mixer" if "ffn" not in p and "side" not in p else ("ffn" if "side" not in p else "side")
+        h = self._add("mixer_norm", x, y, ctx, last == "mixer", gate=z, gate_bias=self.gate_bias.get("mixer_gate"), bias=bias)
+        if "ffn" in p:
+            ffn = p["ffn"]
+            z = ops.linear_parts(h, self.gate["ffn_gate"], ctx.err) if "ffn_gate" in self.gate else None
+            options = dict(leave_rows=True) if getattr(ffn, "leaves_rows", False) else {}
+            if self.joined:
+                options["logits"] = z[..., self.hidden:]
+            y = ffn.forward(h, ctx, **options)
+            h = self._add("ffn_norm", x, y, ctx, last == "ffn", gate=z, gate_bias=self.gate_bias.get("ffn_gate"))
+        if "side" in p:
+            self._add("side_norm", x, p["side"].forward(h, ctx), ctx, True)
+        return x, None
+
+    def _add(self, norm, x, y, ctx, closes, **options):
+        """x += norm(gated y); the new stream in the compute dtype.  `closes`: it is the layer's last addition, whose
+        cast only the next layer's shift would read: it is made with that shift where that is possible."""
+        if isinstance(y, torch.Tensor):
+            y = ops.cast(y, torch.float32)
+        if not closes:
+            return self.p[norm].add_normed(x, y, out_dtype=self.env.dtype, **options)
+        nxt = self.next_block
+        if nxt is None or ctx.max_q_len != 1 or getattr(ctx, "step_cache", None) is None:
+            return self.p[norm].add_normed(x, y, **options)
+        cache = ctx.step_cache(nxt, "shift")
+        h, shifted = self.p[norm].add_normed(x, y, out_dtype=self.env.dtype, next_shift=nxt.p["shift"].ahead(cache), ctx=ctx,
+                                             **options)
+        ctx.shifted_ahead = (nxt, h, shifted)
+        return h

@@ -11,13 +11,14 @@ from .base import Part
 
 
 class TokenEmbedding(Part):
-    """params: vocab_size, hidden_size, alternatives (names that may stand in).
+    """params: vocab_size, hidden_size, alternatives (names that may stand in), scale (absent or 1: none).
     tensors: weight [vocab, hidden].  forward(ctx) -> float32 residual stream [T, hidden] of the
-    step's tokens (`ctx.token_ids`; an embedding that depends on the place reads `ctx.positions`)."""
+    step's tokens, the table's rows times `scale` (`ctx.token_ids`; an embedding that depends on the place reads `ctx.positions`)."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
         self.vocab, self.hidden = int(spec.params["vocab_size"]), int(spec.params["hidden_size"])
+        self.scale = float(spec.params["scale"]) if spec.params.get("scale") is not None else 1.0
         self.weight = None
 
     def tensor_specs(self):
@@ -28,7 +29,7 @@ class TokenEmbedding(Part):
         self.weight = source.get(self.spec.tensors["weight"])
 
     def forward(self, ctx):
-        return ops.embed_gather(ctx.token_ids, self.weight, ctx.err)
+        return ops.embed_gather(ctx.token_ids, self.weight, ctx.err, scale=self.scale)
 
 
 class LMHead(Part):

@@ -12,7 +12,9 @@ one key/value head for all query heads, for prompts and decoded tokens alike.
 
 The queries may go through a latent of their own (`q_rank`): c_q = RMSnorm(W_dq h) with a weight, q = W_uq c_q.  A
 gate per head (`head_gate`) multiplies head h's output by sigmoid(W_g h)_h; it is applied to the head's values before
-the output projection.  The rotation pairs neighbours or halves, as its encoding says.
+the output projection.  The rotation pairs neighbours or halves, as its encoding says, and carries its encoding's
+magnitude.  A softmax may leak into a sink (`sink`): its denominator also holds exp(sink_h), a learned number per head
+that has no key and no value and is not scaled.
 
 A layer may read another layer's cache (`shares_cache`): it has no latent projection of its own and writes
 nothing; the run order names the layer whose rows it reads.
@@ -47,10 +49,10 @@ class LatentAttention(Mixer):
     """params: hidden_size, num_heads, head_dim (unrotated part), rot_dim, value_dim, kv_rank, scale, window
     (0 = all keys), cache_window (the window the cached rows must outlive: the widest of all layers that read
     them; default = window), eps (of the latents' norms), position_encoding (name of a rotary encoding over rot_dim
-    or fewer elements, either layout), shares_cache, q_rank (0: the queries are projected directly), head_gate.
+    or fewer elements, either layout), shares_cache, q_rank (0: the queries are projected directly), head_gate, sink (default False).
     tensors: q [H (d + rot), hidden] (or, with q_rank: dq [q_rank, hidden], dq_norm [q_rank], uq [H (d + rot),
     q_rank]), dkv [kv_rank + rot, hidden], dkv_norm [kv_rank], uk [H d, kv_rank], uv [H dv, kv_rank], o [hidden,
-    H dv], g [H, hidden]."""
+    H dv], g [H, hidden], sink [H]."""
 
     adds_in_place = True
 
@@ -70,9 +72,11 @@ class LatentAttention(Mixer):
             raise ValueError("latent attention: the rotation is wider than rot_dim")
         self.halves = self.rope is not None and not getattr(self.rope, "interleaved", False)
         self.q_rank, self.head_gate = int(p.get("q_rank") or 0), bool(p.get("head_gate"))
+        self.has_sink = bool(p.get("sink"))
+        self.magnitude = float(getattr(self.rope, "magnitude", 1.0)) if self.rope is not None else 1.0
         if (self.q_rank or self.head_gate) and self.shares_cache:
             raise ValueError("latent attention: a layer that reads another's cache has neither a query latent nor a gate")
-        self.w_uq = self.cq_weight = None
+        self.w_uq = self.cq_weight = self.sink = None
         self.w_in = self.w_ukT = self.w_uv = self.w_o = self.c_weight = self._no_rope = None
 
     def tensor_specs(self):
@@ -84,6 +88,8 @@ class LatentAttention(Mixer):
             specs = [TensorSpec(t["q"], (self.H * dq, self.hidden))]
         if self.head_gate:
             specs.append(TensorSpec(t["g"], (self.H, self.hidden)))
+        if self.has_sink:
+            specs.append(TensorSpec(t["sink"], (self.H,), std=1.0))
         if not self.shares_cache:
             specs += [TensorSpec(t["dkv"], (self.rank + self.rot, self.hidden)),
                       TensorSpec(t["dkv_norm"], (self.rank,), init="ones")]
@@ -112,6 +118,8 @@ class LatentAttention(Mixer):
         self.w_ukT = source.get(t["uk"]).view(self.H, self.d, self.rank).transpose(1, 2).contiguous()
         self.w_uv = source.get(t["uv"]).view(self.H, self.dv, self.rank).contiguous()
         self.w_o = source.get(t["o"])
+        if self.has_sink:
+            self.sink = source.get(t["sink"]).float().contiguous()
         self._no_rope = torch.zeros(0, dtype=torch.float32, device=self.env.device)
 
     def weight_bytes(self):
@@ -147,10 +155,11 @@ class LatentAttention(Mixer):
             q_src = proj
         q_plain, q_full = ops.latent_prepare(q_src, self.H, self.d, self.rot, self.rank, self.c_weight, self.eps,
                                              inv_freq, cache.k_pages, ctx, cache.block_table, self.env.dtype,
-                                             write=cache.writes and not self.shares_cache, kv=kv, halves=self.halves)
+                                             write=cache.writes and not self.shares_cache, kv=kv, halves=self.halves,
+                                             magnitude=self.magnitude)
         ops.head_linear(q_plain, self.w_ukT, q_full)
         mixed = ops.latent_attention(q_full, cache.k_pages, ctx, cache.block_table, self.rank, self.scale,
-                                     self.window, self.env.dtype, ctx.plan(LATENT_WORK))
+                                     self.window, self.env.dtype, ctx.plan(LATENT_WORK), sink=self.sink)
         a = torch.empty((T, self.H, self.dv), dtype=self.env.dtype, device=h.device)
         ops.head_linear(mixed, self.w_uv, a)
         a = a.view(T, self.H * self.dv)

@@ -72,6 +72,8 @@ class Model:
                 blk, nxt = self.layers[a].block, self.layers[b].block
                 if hasattr(blk, "set_next_norm") and hasattr(nxt, "first_norm"):
                     blk.set_next_norm(nxt.first_norm())
+                if hasattr(blk, "set_next_block"):
+                    blk.set_next_block(nxt)
         self.keeps_embedding_output = any(getattr(l.block, "needs_embedding_output", False) for l in self.layers)
         self.loaded = False
 
@@ -162,6 +164,9 @@ class Model:
         """`streams`: a list that receives the residual stream [T, hidden] (float32, a copy) behind every entry
         of the run order, for looking at a model layer by layer."""
         ctx.normed_ahead = None           # (norm, its output): made ahead by the block before the one that owns the norm
+        ctx.shifted_ahead = None          # (block, stream, shifted stream): likewise, of the block that owns the shift
+        run_of = {id(self.layers[rs.layer].block): i for i, rs in enumerate(self.order)}
+        ctx.step_cache = lambda block, role: cache.part_cache(run_of[id(block)], role, ctx)
         x = self.embedding.forward(ctx)
         for pe in self.env.position_encodings.values():
             pe.add_to(x, ctx)

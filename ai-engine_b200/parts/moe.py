@@ -107,11 +107,15 @@ class RoutedMoE(FeedForward):
     (+ 1e-20); `route_scale` multiplies them; no tensor `correction`: the choice is made on s itself; a shared
     expert of the same form (`shared_intermediate_size`) runs for every token and is added.
 
+    `score` "softmax_chosen": the router has a bias (tensor `router_bias`), the `top` largest logits are taken and their
+    weights are the softmax over those logits alone (no groups, identity experts, correction or scale).  Without a
+    tensor `gate` an expert is W_down act(W_up h), and `activation` may be any of the plain ones (relu_squared, ...).
+
     params: hidden_size, num_experts (with tensors), identity (default 0), top, intermediate_size, groups
     (default 1), keep (default 1), activation (default "silu"), score (default "softmax"), group_top (default 1),
     normalise (default False), route_scale (default 1), shared_intermediate_size (default 0).  tensors: router
     [num_experts + identity, hidden], correction [num_experts + identity] (optional); gate, up, down as patterns with
-    `{e}` for the expert's index; shared_gate, shared_up, shared_down."""
+    `{e}` for the expert's index; router_bias [num_experts] (score "softmax_chosen"); shared_gate, shared_up, shared_down."""
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -121,19 +125,26 @@ class RoutedMoE(FeedForward):
         self.groups, self.keep = int(p.get("groups") or 1), int(p.get("keep") or 1)
         self.activation = p.get("activation") or "silu"
         total = self.E + self.ident
-        if self.activation != "silu":
-            raise ValueError("routed experts: the experts' activation is silu")
+        self.gated = "gate" in spec.tensors
+        if self.gated and self.activation != "silu":
+            raise ValueError("routed experts: the activation of gated experts is silu")
+        if not self.gated and self.activation not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"routed experts: activation `{self.activation}` is not known ({', '.join(ops.PLAIN_ACTIVATIONS)})")
         if total % self.groups or not 1 <= self.keep <= self.groups or not 1 <= self.top <= total // self.groups * self.keep:
             raise ValueError(f"routed experts: {total} router outputs do not divide into {self.groups} groups of which "
                              f"{self.keep} are kept for {self.top} choices")
         self.score = p.get("score") or "softmax"
-        if self.score not in ("softmax", "sigmoid"):
-            raise ValueError(f"routed experts: score `{self.score}` is not known (softmax, sigmoid)")
+        if self.score not in ("softmax", "sigmoid", "softmax_chosen"):
+            raise ValueError(f"routed experts: score `{self.score}` is not known (softmax, sigmoid, softmax_chosen)")
         self.group_top, self.normalise = int(p.get("group_top") or 1), bool(p.get("normalise"))
         self.route_scale = float(p.get("route_scale") if p.get("route_scale") is not None else 1.0)
         self.has_correction = "correction" in spec.tensors
         self.Fs = int(p.get("shared_intermediate_size") or 0)
-        self.shared = None
+        self.chosen = self.score == "softmax_chosen"
+        if self.chosen and (self.ident or self.groups > 1 or self.has_correction or self.normalise or self.route_scale != 1.0):
+            raise ValueError("routed experts: softmax_chosen weights have no groups, identity experts, correction or scale")
+        self.leaves_rows = not self.ident and not self.Fs
+        self.shared = self.router_bias = None
         if self.Fs:
             from .registry import lookup
             from .spec import PartSpec
@@ -151,9 +162,11 @@ class RoutedMoE(FeedForward):
         specs = [TensorSpec(t["router"], (total, D), std=0.3)]
         if self.has_correction:
             specs.append(TensorSpec(t["correction"], (total,), std=0.05))
+        if self.chosen:
+            specs.append(TensorSpec(t["router_bias"], (total,), std=0.1))
         for e in range(self.E):
-            specs += [TensorSpec(t["gate"].format(e=e), (self.F, D)), TensorSpec(t["up"].format(e=e), (self.F, D)),
-                      TensorSpec(t["down"].format(e=e), (D, self.F))]
+            specs += [TensorSpec(t[n].format(e=e), (self.F, D)) for n in (("gate", "up") if self.gated else ("up",))]
+            specs.append(TensorSpec(t["down"].format(e=e), (D, self.F)))
         return specs + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def load(self, source):
@@ -165,15 +178,18 @@ class RoutedMoE(FeedForward):
             self.w_router = torch.cat([self.w_router, pad], dim=0).contiguous()
         if self.has_correction:
             self.correction = source.get(t["correction"]).float().contiguous()
+        if self.chosen:
+            self.router_bias = source.get(t["router_bias"]).float().contiguous()
         if self.shared is not None:
             self.shared.load(source)
         gu, down = [], []
         for e in range(self.E):
-            gu += [source.get(t["gate"].format(e=e)), source.get(t["up"].format(e=e))]
+            gu += [source.get(t[n].format(e=e)) for n in (("gate", "up") if self.gated else ("up",))]
             down.append(source.get(t["down"].format(e=e)))
         if self.E:
             dt = torch.float32 if any(w.dtype == torch.float32 for w in gu + down) else gu[0].dtype
-            self.w_gu = torch.stack([w.to(dt) for w in gu]).view(self.E, 2 * self.F, self.hidden).contiguous()
+            # [E, (gate rows and) up rows, hidden]
+            self.w_gu = torch.stack([w.to(dt) for w in gu]).view(self.E, (2 if self.gated else 1) * self.F, self.hidden).contiguous()
             self.w_down = torch.stack([w.to(dt) for w in down]).contiguous()              # [E, hidden, F]
 
     def weight_bytes(self):
@@ -182,18 +198,25 @@ class RoutedMoE(FeedForward):
             + (self.shared.weight_bytes() if self.shared is not None else 0)
 
     def flops(self, tokens, keys=0.0):
-        return 2.0 * tokens * self.hidden * (3 * self.top * self.F + self.E + self.ident) \
+        return 2.0 * tokens * self.hidden * ((3 if self.gated else 2) * self.top * self.F + self.E + self.ident) \
             + (self.shared.flops(tokens, keys) if self.shared is not None else 0.0)
 
-    def forward(self, h, ctx):
+    def router_weight(self):
+        return self.w_router
+
+    def forward(self, h, ctx, logits=None, leave_rows=False):
         # the router in float32 on the sublayer's input as the experts see it: products of bfloat16 values are exact
         # in float32, so the tensor-core product with float32 sums is a float32 product of those inputs
-        if h.dtype == torch.bfloat16 and self.w_router.dtype == torch.bfloat16:
+        if logits is not None:
+            pass
+        elif h.dtype == torch.bfloat16 and self.w_router.dtype == torch.bfloat16:
             logits = ops.linear(h, self.w_router, torch.float32, ctx.err)[:, :self.E + self.ident]
         else:
             logits = ops.gemm_f32(ops.cast(h, torch.float32), self.w_router)
-        ids, weights = ops.route_topk(logits, self.correction, self.groups, self.keep, self.top, score=self.score,
-                                      group_top=self.group_top, normalise=self.normalise, weight_scale=self.route_scale)
+        if self.chosen:
+            ids, weights = ops.route_chosen(logits, self.router_bias, self.E, self.top)
+        else:
+            ids, weights = self._grouped_choice(logits)
         shared = self.shared.forward(h, ctx) if self.shared is not None else None
         if not self.E:
             y = torch.zeros((1, self.hidden), dtype=torch.float32, device=h.device)
@@ -201,6 +224,15 @@ class RoutedMoE(FeedForward):
             return ops.expert_combine_weighted(y, pair_row, weights, h, shared)
         row_token, pair_row, tile_expert = ops.expert_plan(None, ids, self.E, ctx.err, identity=self.ident)
         gu = ops.grouped_linear(h, self.w_gu, tile_expert, torch.float32, ctx.err, row_src=row_token)
-        act = ops.clamped_glu(gu, self.F, float("inf"), 1.0, 0.0, self.env.dtype)       # silu(gate) * up
+        if self.gated:
+            act = ops.clamped_glu(gu, self.F, float("inf"), 1.0, 0.0, self.env.dtype)       # silu(gate) * up
+        else:
+            act = ops.activate(gu, self.activation, self.env.dtype)
         y = ops.grouped_linear(act, self.w_down, tile_expert, torch.float32, ctx.err)
+        if leave_rows and self.leaves_rows:
+            return ops.ExpertRows(y, pair_row, weights)
         return ops.expert_combine_weighted(y, pair_row, weights, h, shared)
+
+    def _grouped_choice(self, logits):
+        return ops.route_topk(logits, self.correction, self.groups, self.keep, self.top, score=self.score,
+                              group_top=self.group_top, normalise=self.normalise, weight_scale=self.route_scale)

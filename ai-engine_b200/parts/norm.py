@@ -38,6 +38,13 @@ class RMSNorm(Norm):
         return ops.add_rmsnorm(x, delta, self.weight, self.eps, self.out_dtype, rows=rows,
                                write_back=write_back)
 
+    def add_normed(self, x, y, **options):
+        """x += norm(y) in place, for a norm on a sublayer's output; the options (a gate on y, a bias, the new stream in
+        a compute dtype, ...) and the result are those of `ops.gated_norm_add`."""
+        if self.weight.dtype != torch.float32:
+            self.weight = self.weight.float().contiguous()
+        return ops.gated_norm_add(x, y, self.weight, self.eps, **options)
+
 
 class DynamicTanh(Norm):
     """A norm that computes no mean and no variance: y = tanh(alpha x) * w + b, element by element in float32.

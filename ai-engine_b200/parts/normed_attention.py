@@ -50,6 +50,8 @@ class NormedGatedAttention(Mixer):
         self.rope = env.position_encodings[pe] if pe else None
         if self.rope is not None and self.rope.rot_dim > self.d:
             raise ValueError("attention: the rotation is wider than a head")
+        if self.rope is not None and getattr(self.rope, "magnitude", 1.0) != 1.0:
+            raise ValueError("attention: its kernels rotate without a magnitude; a yarn encoding is not taken")
         self.value_mix = p.get("value_mix")
         if self.value_mix not in (None, "source", "mix"):
             raise ValueError(f"attention: value_mix `{self.value_mix}` is not known (source, mix)")
