@@ -82,4 +82,4 @@ def named(read: Callable, where: str):
     try:
         return read()
     except ConfigError as e:
-        raise ConfigError(str(e).replace("config.json: ", f"config.json: {where}", 1)) from None
+        raise ConfigError(str(e).replace("config.json: ", f"config.json: in {where.rstrip('.')}: ", 1)) from None

@@ -17,6 +17,7 @@
 #include "common.cuh"
 
 #define LAT_CHUNK 128
+#define LAT_PREP 128       // threads that share the sum over a latent
 
 // element i of a rot-wide vector x after the rotation by `pos`
 __device__ __forceinline__ float latent_rotated(const float* x, int i, int half, int halves, int pos,
@@ -62,7 +63,8 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld, in
     if (!has_kv) return;
     const float* z = kv ? kv + (size_t)t * ld_kv : row + H * dq;
     float ss = 0.f;
-    for (int i = tid; i < rank; i += blockDim.x) ss += z[i] * z[i];
+    if (tid < LAT_PREP)                                 // always the same threads: a latent's bits do not depend on the step
+        for (int i = tid; i < rank; i += LAT_PREP) ss += z[i] * z[i];
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)rank + eps);
     const int pidx = pos / P;
@@ -84,8 +86,9 @@ extern "C" int aie_latent_prepare(const float* proj, int ld, int T, int H, int d
                                   unsigned* err, const float* kv, int ld_kv, int halves, float mag, cudaStream_t st) {
     if (T <= 0) return 0;
     if (rot_dims % 2 || rot_dims > rot || H <= 0 || d < 0 || rank <= 0) return AIE_BAD_ARG;
+    const int threads = T <= 2 * aie_sm_count() ? 1024 : LAT_PREP;      // few tokens: a block has an SM to itself
 #define GO(A, C)                                                                                                      \
-    latent_prepare_kernel<A, C><<<T, 128, 0, st>>>(proj, ld, H, d, rot, rank, rot_dims, has_kv, c_weight, eps, inv_freq, \
+    latent_prepare_kernel<A, C><<<T, threads, 0, st>>>(proj, ld, H, d, rot, rank, rot_dims, has_kv, c_weight, eps, inv_freq, \
                                                    (A*)q_plain, q_full, (C*)pages, positions, token_req, block_table,  \
                                                    bt_width, num_pages, P, err, kv, ld_kv, halves, mag)
     if (q_dtype == AIE_F32 && cache_dtype == AIE_F32) GO(float, float);

@@ -233,23 +233,39 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
     }
 }
 
-// out[t, h] = sum_p w_p O_p / sum_p w_p l_p with w_p = exp(m_p - max m), parts in order
+// out[t, h] = sum_p w_p O_p / sum_p w_p l_p with w_p = exp(m_p - max m), parts in order.  The first warp makes the
+// weights of all parts (at most 64), then every thread adds its column with several parts' loads in flight.
 __global__ void latent_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                    bf16* __restrict__ out, int splits, int rank) {
+    __shared__ float w_s[64];
+    __shared__ float inv_s;
     const size_t th = blockIdx.x;
     const float* ml = part_ml + th * splits * 2;
-    float mx = -INFINITY;
-    for (int p = 0; p < splits; ++p)
-        if (ml[2 * p + 1] > 0.f) mx = fmaxf(mx, ml[2 * p]);
-    float den = 0.f;
-    for (int p = 0; p < splits; ++p)
-        if (ml[2 * p + 1] > 0.f) den += expf(ml[2 * p] - mx) * ml[2 * p + 1];
-    const float inv = den > 0.f ? 1.0f / den : 0.f;
-    for (int c = threadIdx.x; c < rank; c += blockDim.x) {
-        float acc = 0.f;
-        for (int p = 0; p < splits; ++p)
-            if (ml[2 * p + 1] > 0.f) acc = fmaf(expf(ml[2 * p] - mx), part_o[(th * splits + p) * rank + c], acc);
-        out[th * rank + c] = __float2bfloat16_rn(acc * inv);
+    if (threadIdx.x < 32) {
+        const int a = threadIdx.x, b = a + 32;
+        const float la = a < splits ? ml[2 * a + 1] : 0.f, lb = b < splits ? ml[2 * b + 1] : 0.f;
+        const float ma = la > 0.f ? ml[2 * a] : -INFINITY, mb = lb > 0.f ? ml[2 * b] : -INFINITY;
+        const float mx = warp_max(fmaxf(ma, mb));
+        const float wa = la > 0.f ? expf(ma - mx) : 0.f, wb = lb > 0.f ? expf(mb - mx) : 0.f;
+        w_s[a] = wa;
+        w_s[b] = wb;
+        const float den = warp_sum(wa * la + wb * lb);
+        if (a == 0) inv_s = den > 0.f ? 1.0f / den : 0.f;
+    }
+    __syncthreads();
+    const float inv = inv_s;
+    for (int c = threadIdx.x * 4; c < rank; c += blockDim.x * 4) {
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int p = 0; p < splits; ++p) {                 // an empty part wrote zeros and weighs nothing
+            const float4 v = *reinterpret_cast<const float4*>(part_o + (th * splits + p) * rank + c);
+            const float w = w_s[p];
+            acc.x = fmaf(w, v.x, acc.x);
+            acc.y = fmaf(w, v.y, acc.y);
+            acc.z = fmaf(w, v.z, acc.z);
+            acc.w = fmaf(w, v.w, acc.w);
+        }
+        store4<bf16>(out + th * rank + c, make_float4(acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv));
     }
 }
 
@@ -292,5 +308,78 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     if (splits > 1) latent_join_kernel<<<T * H, 128, 0, st>>>(part_o, part_ml, (bf16*)out, splits, rank);
+    AIE_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------------------
+// Per-head products of small steps: out[t, h, n] = sum_k w[h, n, k] x[t, h, k], bfloat16 operands, float32 sums.  What
+// bounds them is the stream of the weights.  A CTA of four warps owns 16 rows n of one head for all tokens; the warps
+// take every fourth block of 32 k and are joined through shared memory.  A thread reads its operands 16 bytes at a
+// time: the eight consecutive k it loads stand for the pairs that two mma.sync k16 steps want of it, in weights and
+// activations alike, and a sum over k has no order to keep.
+#define HL_TOKENS 64
+
+template <int NT, typename O>       // token tiles of 8
+__global__ void __launch_bounds__(128)
+head_linear_small_kernel(const bf16* __restrict__ x, long long xt, long long xh, const bf16* __restrict__ w,
+                         O* __restrict__ out, long long ot, long long oh, int T, int N, int K) {
+    __shared__ float part[4][16][NT * 8 + 1];
+    const int h = blockIdx.y, n0 = blockIdx.x * 16;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = lane >> 2, q = lane & 3;
+    const bf16* wh = w + (size_t)h * N * K;
+    const bool on0 = n0 + row < N, on1 = n0 + row + 8 < N;
+    const bf16* w0 = wh + (size_t)(on0 ? n0 + row : 0) * K + q * 8;
+    const bf16* w1 = wh + (size_t)(on1 ? n0 + row + 8 : 0) * K + q * 8;
+    float acc[NT][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll 4
+    for (int k = warp * 32; k < K; k += 128) {
+        const uint4 a0 = on0 ? *reinterpret_cast<const uint4*>(w0 + k) : zero;
+        const uint4 a1 = on1 ? *reinterpret_cast<const uint4*>(w1 + k) : zero;
+        const unsigned f0[4] = {a0.x, a1.x, a0.y, a1.y}, f1[4] = {a0.z, a1.z, a0.w, a1.w};
+#pragma unroll
+        for (int i = 0; i < NT; ++i) {
+            const int t = i * 8 + row;
+            const uint4 b = t < T ? *reinterpret_cast<const uint4*>(x + t * xt + h * xh + k + q * 8) : zero;
+            mma16816(acc[i], f0, b.x, b.y);
+            mma16816(acc[i], f1, b.z, b.w);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) part[warp][row + (e >> 1) * 8][i * 8 + q * 2 + (e & 1)] = acc[i][e];
+    __syncthreads();
+    for (int i = tid; i < 16 * NT * 8; i += 128) {
+        const int n = i & 15, t = i >> 4;
+        if (t < T && n0 + n < N)
+            out[t * ot + h * oh + n0 + n] = from_f32<O>((part[0][n][t] + part[1][n][t]) + (part[2][n][t] + part[3][n][t]));
+    }
+}
+
+// x rows xt apart (tokens) and xh apart (heads), out likewise (elements); w [H, N, K] bfloat16.  T <= 64, K a multiple of
+// 32, x and its strides aligned to 16 bytes (else AIE_UNSUPPORTED).
+extern "C" int aie_head_linear_small(const void* x, long long xt, long long xh, const void* w, void* out, int out_dtype,
+                                     long long ot, long long oh, int T, int H, int N, int K, cudaStream_t st) {
+    if (T <= 0) return 0;
+    if (T > HL_TOKENS || K % 32 || xt % 8 || xh % 8 || ((size_t)x & 15) || ((size_t)w & 15) || H > 65535) return AIE_UNSUPPORTED;
+    const dim3 grid((N + 15) / 16, H);
+#define GO(NT, O) head_linear_small_kernel<NT, O><<<grid, 128, 0, st>>>((const bf16*)x, xt, xh, (const bf16*)w, (O*)out, ot, oh, T, N, K)
+#define GO_O(O)                                                                                                       \
+    if (T <= 8) GO(1, O);                                                                                             \
+    else if (T <= 16) GO(2, O);                                                                                       \
+    else if (T <= 32) GO(4, O);                                                                                       \
+    else GO(8, O)
+    if (out_dtype == AIE_F32) {
+        GO_O(float);
+    } else if (out_dtype == AIE_BF16) {
+        GO_O(bf16);
+    } else {
+        return AIE_BAD_ARG;
+    }
+#undef GO_O
+#undef GO
     AIE_LAUNCH_CHECK();
 }

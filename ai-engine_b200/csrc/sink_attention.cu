@@ -196,6 +196,52 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
     }
 }
 
+// The same for heads that are normed one by one, not rotated and not mixed: a warp per head of q, k or v, a head's
+// elements in registers (d <= 256).
+template <typename A>
+__global__ void __launch_bounds__(256)
+head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias,
+                           const float* __restrict__ q_w, const float* __restrict__ k_w, float eps, A* __restrict__ q_out,
+                           A* __restrict__ pages, const int* __restrict__ positions, const int* __restrict__ token_req,
+                           const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
+                           int e, int maps, int write, unsigned* err) {
+    const int t = blockIdx.x, lane = threadIdx.x & 31;
+    const int K = G * maps, nq = H * d, nk = K * d;
+    const int hh = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);      // heads of q, then of k, then of v
+    if (hh >= H + K + G || (hh >= H && !write)) return;
+    const bool is_v = hh >= H + K;
+    const int n = is_v ? e : d;
+    const int at = is_v ? nq + nk + (hh - H - K) * e : hh * d;
+    const float* row = proj + (size_t)t * ld + at;
+    const float* b = bias ? bias + at : nullptr;
+    A* dst = q_out + (size_t)t * nq + hh * d;
+    if (hh >= H) {
+        const int pos = positions[t], pidx = pos / P;
+        const int page = (pos >= 0 && pidx < bt_width) ? block_table[(size_t)token_req[t] * bt_width + pidx] : -1;
+        if (page < 0 || page >= num_pages) {
+            if (lane == 0) atomicOr(err, AIE_DEV_PAGE_OOB);
+            return;
+        }
+        const int k = hh - H, g = is_v ? k - K : k / maps;
+        dst = pages + (((size_t)page * G + g) * P + (pos - pidx * P)) * (maps * d + e) + (is_v ? maps * d : (k % maps) * d);
+    }
+    float x[8], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int c = lane + 32 * i;
+        x[i] = c < n ? row[c] + (b ? b[c] : 0.f) : 0.f;
+        ss += x[i] * x[i];
+    }
+    float inv = 1.f;
+    const float* w = is_v ? nullptr : (hh < H ? q_w : k_w);
+    if (w) inv = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int c = lane + 32 * i;
+        if (c < n) dst[c] = from_f32<A>(w ? (x[i] * inv) * w[c] : x[i]);
+    }
+}
+
 extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* bias, const float* q_w, const float* k_w,
                                        float eps, const float* inv_freq, int rot_dims, int halves, const float* mix_from,
                                        const float* lambda, float* v_keep, void* q_out, void* pages, int dtype,
@@ -207,6 +253,16 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
     if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || rot_dims < 0 || rot_dims > d || rot_dims % 2 ||
         (mix_from && !lambda) || (q_w && !k_w) || (rot_dims > 0 && !inv_freq))
         return AIE_BAD_ARG;
+    if ((per_head || !q_w) && rot_dims == 0 && !mix_from && !v_keep && d <= 256 && e <= 256) {
+        const dim3 grid(T, (H + G * maps + G + 7) / 8);
+        if (dtype == AIE_F32)
+            head_normed_prepare_kernel<float><<<grid, 256, 0, stream>>>(proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+        else if (dtype == AIE_BF16)
+            head_normed_prepare_kernel<bf16><<<grid, 256, 0, stream>>>(proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+        else
+            return AIE_BAD_ARG;
+        AIE_LAUNCH_CHECK();
+    }
     const size_t smem = ((size_t)(H + G * maps) * d + 32) * sizeof(float);
     if (smem > 200 * 1024) return AIE_UNSUPPORTED;
 #define AIE_NAP(A)                                                                                                    \

@@ -600,6 +600,15 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Te
             else:
                 torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=dst)
         return out
+    if (T <= 64 and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and K % 32 == 0 and x.stride(0) % 8 == 0
+            and x.stride(1) % 8 == 0 and x.data_ptr() % 16 == 0):
+        # few tokens: a stream of the heads' weights through the tensor cores
+        with region("head_linear", _nb(w) + T * H * (K * 2 + N * out.element_size()), 2.0 * T * H * N * K):
+            check(library("latent_attention_tc.cu").aie_head_linear_small(
+                _p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _p(w), _p(out), c_int(dtype_code(out)),
+                c_longlong(out.stride(0)), c_longlong(out.stride(1)), c_int(T), c_int(H), c_int(N), c_int(K), _stream()),
+                "head_linear")
+        return out
     return gemm_f32_ex(x, w, out, T, N, K, x.stride(0), out.stride(0), batch=H, a_bs=x.stride(1), w_bs=N * K,
                        c_bs=out.stride(1))
 

@@ -132,6 +132,23 @@ def fokisun_shape(width, layers=8):
                 layers=out)
 
 
+def vatazen_shape(width, layers=8):
+    """A Vatazen configuration with layers of the sizes real models of its kind have: latent-attention heads of 128 + 64
+    rotated with a latent of width / 4 (256 to 512) under a window of 1,024, positions stretched by 8; differential
+    heads of two maps of 64 over values of 128 (a quarter of them key/value heads) in chunks of 2,048; experts without a
+    gate of 3 / 4 width (top 4 of 32); a token input of width / 16 per layer.  The pattern (latent attention,
+    differential attention) repeats."""
+    H = width // 128
+    lat = dict(type="latent_attention", mixer=dict(
+        heads=H, dim=128, rot_dim=64, vdim=128, kv_rank=min(512, max(256, width // 4)), scale=192 ** -0.5, mask=dict(size=1024),
+        rot=dict(base=500000.0, dims=64, scaling=dict(factor=8.0, original=4096, fast=32.0, slow=1.0))))
+    att = dict(type="attention", mixer=dict(heads=H, kv_heads=max(1, H // 4), dim=64, vdim=128, scale=64 ** -0.5, diff=0.2,
+                                            mask=dict(size=2048)))
+    moe = dict(kind="moe", expert=dict(ff=3 * width // 4), router=dict(experts=32, top=4))
+    return dict(architecture="Vatazen", vocab=32000, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                token_side=dict(dim=width // 16), layers=[dict((lat, att)[i % 2], mlp=moe) for i in range(layers)])
+
+
 def llama_like(width, layers=8):
     """The closest existing model at equal size: the same width, layers, heads of 128 (a quarter of them kv heads)
     and a feed-forward of 3 x width, which is what a Pifutar token uses (4 experts of width / 2 + the shared one)."""
@@ -674,10 +691,10 @@ def main():
                     help="time one part only and print its numbers (for profiling)")
     ap.add_argument("--profile", action="store_true",
                     help="CUDA-event time, bytes, flops and roofline fraction per class of kernel (eager launches)")
-    ap.add_argument("--shape", choices=["8b", "1b", "3b"] + [f"{m}-{w}" for m in ("pifutar", "zupitar", "tizodra", "fokisun", "llama") for w in WIDTHS],
+    ap.add_argument("--shape", choices=["8b", "1b", "3b"] + [f"{m}-{w}" for m in ("pifutar", "zupitar", "tizodra", "fokisun", "vatazen", "llama") for w in WIDTHS],
                     default="8b",
                     help="layer sizes for --profile and --only decode|prefill (the headline run is always the 8B shape); "
-                         "pifutar-1k|2k|4k, zupitar-1k|2k|4k, tizodra-1k|2k|4k, fokisun-1k|2k|4k: those designs at that width, llama-1k|2k|4k: Llama at equal size beside them "
+                         "pifutar-1k|2k|4k, zupitar-1k|2k|4k, tizodra-1k|2k|4k, fokisun-1k|2k|4k, vatazen-1k|2k|4k: those designs at that width, llama-1k|2k|4k: Llama at equal size beside them "
                          "(8 layers unless --layers says otherwise)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="cached tokens per request for --profile / --only decode")
     ap.add_argument("--skip-workloads", action="store_true", help="leave the 1B and 3B serving workloads out of `points`")
@@ -724,7 +741,7 @@ def main():
     if "-" in a.shape and (a.profile or a.only):
         family, w = a.shape.split("-")
         layers = a.layers if a.layers != LLAMA3_8B["num_hidden_layers"] else 8
-        cfg = dict(pifutar=pifutar_shape, zupitar=zupitar_shape, tizodra=tizodra_shape, fokisun=fokisun_shape, llama=llama_like)[family](WIDTHS[w], layers)
+        cfg = dict(pifutar=pifutar_shape, zupitar=zupitar_shape, tizodra=tizodra_shape, fokisun=fokisun_shape, vatazen=vatazen_shape, llama=llama_like)[family](WIDTHS[w], layers)
     else:
         cfg = dict({"8b": LLAMA3_8B, "1b": LLAMA32_1B, "3b": LLAMA32_3B}.get(a.shape, LLAMA3_8B) if (a.profile or a.only) else LLAMA3_8B)
         if a.layers != LLAMA3_8B["num_hidden_layers"] or a.shape == "8b":

@@ -150,3 +150,36 @@ def test_groups_by_what_parts_ask_for():
     assert c.book.group(1).window == 32
     with pytest.raises(ValueError):
         PagedCache([CacheNeed(1, "mixer", None, None, 0)], 8, 10, 2, 64, None, allocate=False)
+
+
+def test_chunks_give_pages_back_at_their_edge():
+    """A group in chunks of 20 on pages of 8: while a chunk fills every page of it is kept, also the one its first
+    token shares with the chunk before; at the first token of the next chunk all earlier pages go."""
+    h = host()
+    g = h.GroupSpec(8, 7, 0, 0, 20)
+    assert g.chunk == 20
+    c = h.CacheManager([g], 2, 64)
+    s = c.admit()
+    assert c.ensure(s, 19) and c.advance(s, 19) == 0       # the query at 19 still reads from 0 on
+    assert c.ensure(s, 20) and c.advance(s, 20) == 2       # queries from 20 on read [20, ..): pages 0, 1 (keys 0 .. 15) go
+    assert c.pages(0, s)[:2] == [-1, -1] and c.first_live(0, s) == 2
+    assert c.ensure(s, 39) and c.advance(s, 39) == 0 and c.pages_in_use(0) == 3
+    assert c.ensure(s, 40) and c.advance(s, 40) == 3 and c.pages_in_use(0) == 0
+    for n in range(41, 200):                               # never more than the pages a chunk touches
+        assert c.ensure(s, n), n
+        c.advance(s, n)
+        assert c.pages_in_use(0) <= 4
+        c.check_invariants()
+    c.finish(s)
+    assert c.free_pages(0) == 7
+    with pytest.raises(Exception, match="not both"):
+        h.CacheManager([h.GroupSpec(8, 4, 16, 0, 16)], 1, 4)
+
+
+def test_bytes_read_in_chunks():
+    kv = KVRequest(2, 24, planes=1, chunk=32)
+    from ai_engine_b200.parts import CacheNeed
+    import torch
+    c = PagedCache([CacheNeed(0, "mixer", kv)], page_size=8, num_pages=10, max_seqs=1, max_seq_len=64, dtype=torch.bfloat16,
+                   allocate=False)
+    assert c.kv_bytes_read(31) == 32 * 48 * 2 and c.kv_bytes_read(32) == 48 * 2 and c.book.group(0).chunk == 32
