@@ -453,6 +453,40 @@ __global__ void activate_kernel(const I* __restrict__ z, O* __restrict__ out, si
         for (size_t j = i; j < n; ++j) out[j] = from_f32<O>(plain_act(to_f32<I>(z[j]), act));
 }
 
+// the same on the rows r of z [n, F] whose rows[r] >= 0 (the others, padding of a grouping, are left as they are)
+template <typename I, typename O>
+__global__ void activate_rows_kernel(const I* __restrict__ z, const int* __restrict__ rows, O* __restrict__ out, int F, int act) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r = blockIdx.x;
+    if (rows[r] < 0) return;
+    const I* a = z + (size_t)r * F;
+    O* b = out + (size_t)r * F;
+    if (F % 4 == 0) {
+        for (int c = threadIdx.x * 4; c < F; c += blockDim.x * 4) {
+            float4 v = load4<I>(a + c);
+            v.x = plain_act(v.x, act); v.y = plain_act(v.y, act); v.z = plain_act(v.z, act); v.w = plain_act(v.w, act);
+            store4<O>(b + c, v);
+        }
+    } else {
+        for (int c = threadIdx.x; c < F; c += blockDim.x) b[c] = from_f32<O>(plain_act(to_f32<I>(a[c]), act));
+    }
+}
+
+extern "C" int aie_activate_rows(const void* z, int in_dtype, const int* rows, void* out, int out_dtype, int n, int F, int act,
+                                 cudaStream_t stream) {
+    if (n <= 0) return 0;
+    if (act < 0 || act > 3 || F <= 0) return AIE_BAD_ARG;
+    const dim3 threads(F >= 1024 ? 256 : 128);
+    if (in_dtype == AIE_F32 && out_dtype == AIE_F32)
+        launch_pdl(activate_rows_kernel<float, float>, dim3(n), threads, 0, stream, (const float*)z, rows, (float*)out, F, act);
+    else if (in_dtype == AIE_F32 && out_dtype == AIE_BF16)
+        launch_pdl(activate_rows_kernel<float, bf16>, dim3(n), threads, 0, stream, (const float*)z, rows, (bf16*)out, F, act);
+    else
+        return AIE_BAD_ARG;
+    AIE_LAUNCH_CHECK();
+}
+
 extern "C" int aie_activate(const void* z, int in_dtype, void* out, int out_dtype, long long n, int act,
                             cudaStream_t stream) {
     if (n <= 0) return 0;

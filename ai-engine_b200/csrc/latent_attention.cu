@@ -46,6 +46,8 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int ld, in
                                       const int* __restrict__ block_table, int bt_width, int num_pages, int P,
                                       unsigned* err, const float* __restrict__ kv, int ld_kv, int halves, float mag) {
     __shared__ float red[32];
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x, tid = threadIdx.x;
     const float* row = proj + (size_t)t * ld;
     const int pos = positions[t];
@@ -88,7 +90,7 @@ extern "C" int aie_latent_prepare(const float* proj, int ld, int T, int H, int d
     if (rot_dims % 2 || rot_dims > rot || H <= 0 || d < 0 || rank <= 0) return AIE_BAD_ARG;
     const int threads = T <= 2 * aie_sm_count() ? 1024 : LAT_PREP;      // few tokens: a block has an SM to itself
 #define GO(A, C)                                                                                                      \
-    latent_prepare_kernel<A, C><<<T, threads, 0, st>>>(proj, ld, H, d, rot, rank, rot_dims, has_kv, c_weight, eps, inv_freq, \
+    launch_pdl(latent_prepare_kernel<A, C>, dim3(T), dim3(threads), 0, st, proj, ld, H, d, rot, rank, rot_dims, has_kv, c_weight, eps, inv_freq, \
                                                    (A*)q_plain, q_full, (C*)pages, positions, token_req, block_table,  \
                                                    bt_width, num_pages, P, err, kv, ld_kv, halves, mag)
     if (q_dtype == AIE_F32 && cache_dtype == AIE_F32) GO(float, float);

@@ -39,6 +39,8 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
     float* l_all = m_all + TQ * LT_ROWS;                          // [TQ][16] running sum
     float* c_all = l_all + TQ * LT_ROWS;                          // [TQ][16] correction of this chunk
 
+    pdl_launch_dependents();
+    pdl_wait();
     const int row = tiles[2 * blockIdx.x], off = tiles[2 * blockIdx.x + 1];
     const int h0 = blockIdx.y * LT_ROWS, part = blockIdx.z;
     const int tid = threadIdx.x, tq = tid / LT_THREADS, ltid = tid % LT_THREADS, warp = (tid >> 5) & 3, lane = tid & 31;
@@ -239,6 +241,8 @@ __global__ void latent_join_kernel(const float* __restrict__ part_o, const float
                                    bf16* __restrict__ out, int splits, int rank) {
     __shared__ float w_s[64];
     __shared__ float inv_s;
+    pdl_launch_dependents();
+    pdl_wait();
     const size_t th = blockIdx.x;
     const float* ml = part_ml + th * splits * 2;
     if (threadIdx.x < 32) {
@@ -291,7 +295,7 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
     {                                                                                                                 \
         auto kern = latent_attention_tc_kernel<CWV, TQV>;                                                             \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
-        kern<<<grid, LT_THREADS * TQV, smem, st>>>(q_full, (const bf16*)pages, (bf16*)out, part_o, part_ml, tiles,    \
+        launch_pdl(kern, grid, dim3(LT_THREADS * TQV), smem, st, q_full, (const bf16*)pages, (bf16*)out, part_o, part_ml, tiles,    \
                                                    q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, H,   \
                                                    dk, window, scale, splits, sink, err);                                   \
     }
@@ -307,7 +311,7 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
 #undef GO1
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
-    if (splits > 1) latent_join_kernel<<<T * H, 128, 0, st>>>(part_o, part_ml, (bf16*)out, splits, rank);
+    if (splits > 1) launch_pdl(latent_join_kernel, dim3(T * H), dim3(128), 0, st, part_o, part_ml, (bf16*)out, splits, rank);
     AIE_LAUNCH_CHECK();
 }
 
@@ -324,6 +328,8 @@ __global__ void __launch_bounds__(128)
 head_linear_small_kernel(const bf16* __restrict__ x, long long xt, long long xh, const bf16* __restrict__ w,
                          O* __restrict__ out, long long ot, long long oh, int T, int N, int K) {
     __shared__ float part[4][16][NT * 8 + 1];
+    pdl_launch_dependents();
+    pdl_wait();
     const int h = blockIdx.y, n0 = blockIdx.x * 16;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = lane >> 2, q = lane & 3;
     const bf16* wh = w + (size_t)h * N * K;
@@ -366,7 +372,7 @@ extern "C" int aie_head_linear_small(const void* x, long long xt, long long xh, 
     if (T <= 0) return 0;
     if (T > HL_TOKENS || K % 32 || xt % 8 || xh % 8 || ((size_t)x & 15) || ((size_t)w & 15) || H > 65535) return AIE_UNSUPPORTED;
     const dim3 grid((N + 15) / 16, H);
-#define GO(NT, O) head_linear_small_kernel<NT, O><<<grid, 128, 0, st>>>((const bf16*)x, xt, xh, (const bf16*)w, (O*)out, ot, oh, T, N, K)
+#define GO(NT, O) launch_pdl(head_linear_small_kernel<NT, O>, grid, dim3(128), 0, st, (const bf16*)x, xt, xh, (const bf16*)w, (O*)out, ot, oh, T, N, K)
 #define GO_O(O)                                                                                                       \
     if (T <= 8) GO(1, O);                                                                                             \
     else if (T <= 16) GO(2, O);                                                                                       \

@@ -415,6 +415,8 @@ __global__ void expert_plan_kernel(const int* __restrict__ ids, const int* __res
                                    int E, int ident, int tile, int n_tiles, int* __restrict__ row_token, int* __restrict__ pair_row,
                                    int* __restrict__ tile_expert, unsigned* err) {
     extern __shared__ int sh[];
+    pdl_launch_dependents();
+    pdl_wait();
     int* count = sh;            // [E]
     int* start = sh + E;        // [E]
     int* cursor = sh + 2 * E;   // [E]
@@ -435,13 +437,24 @@ __global__ void expert_plan_kernel(const int* __restrict__ ids, const int* __res
         atomicAdd(&count[e], 1);
     }
     __syncthreads();
-    if (tid == 0) {
-        int at = 0;
-        for (int e = 0; e < E; ++e) {
-            start[e] = at * tile;
-            const int nt = (count[e] + tile - 1) / tile;
-            for (int i = 0; i < nt && at + i < n_tiles; ++i) tile_expert[at + i] = e;
-            at += nt;
+    if (tid < 32) {                          // the first warp adds up the tiles of the experts before, 32 at a time
+        int base = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + tid;
+            const int nt = e < E ? (count[e] + tile - 1) / tile : 0;
+            int at = nt;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int v = __shfl_up_sync(0xffffffffu, at, o);
+                if (tid >= o) at += v;
+            }
+            const int total = __shfl_sync(0xffffffffu, at, 31);
+            at += base - nt;
+            if (e < E) {
+                start[e] = at * tile;
+                for (int i = 0; i < nt && at + i < n_tiles; ++i) tile_expert[at + i] = e;
+            }
+            base += total;
         }
     }
     __syncthreads();
@@ -464,7 +477,7 @@ extern "C" int aie_expert_plan(const int* ids, const int* table, int T, int V, i
     if (T <= 0) return 0;
     if (top <= 0 || E <= 0 || tile <= 0 || (long long)n_tiles * tile < (long long)T * top) return AIE_BAD_ARG;
     if ((size_t)3 * E * sizeof(int) > 40000) return AIE_UNSUPPORTED;
-    expert_plan_kernel<<<1, 1024, 3 * E * sizeof(int), st>>>(ids, table, T, V, top, E, ident, tile, n_tiles, row_token, pair_row,
+    launch_pdl(expert_plan_kernel, dim3(1), dim3(1024), 3 * E * sizeof(int), st, ids, table, T, V, top, E, ident, tile, n_tiles, row_token, pair_row,
                                                               tile_expert, err);
     AIE_LAUNCH_CHECK();
 }
@@ -495,21 +508,37 @@ extern "C" int aie_expert_combine(const float* y, const int* pair_row, int top, 
     AIE_LAUNCH_CHECK();
 }
 
-// out[r] = src[rows[r]] (zeros where rows[r] < 0): the step's rows in the order of a grouping
+// out[r] = src[rows[r]]: the step's rows in the order of a grouping.  Where rows[r] < 0 the row is zeros, or, without
+// `zero_fill`, left as it is (padding whose products nobody reads).  Rows go 16 bytes a thread where they are aligned.
 template <typename T>
-__global__ void gather_rows_kernel(const T* __restrict__ src, const int* __restrict__ rows, T* __restrict__ out, int D) {
+__global__ void gather_rows_kernel(const T* __restrict__ src, const int* __restrict__ rows, T* __restrict__ out, int D,
+                                   int zero_fill, int vec) {
+    pdl_launch_dependents();
+    pdl_wait();
     const int r = blockIdx.x, s = rows[r];
+    if (s < 0 && !zero_fill) return;
+    if (vec) {
+        const int n = D * (int)sizeof(T) / 16;
+        const uint4* a = reinterpret_cast<const uint4*>(src + (size_t)(s >= 0 ? s : 0) * D);
+        uint4* b = reinterpret_cast<uint4*>(out + (size_t)r * D);
+        for (int c = threadIdx.x; c < n; c += blockDim.x) b[c] = s >= 0 ? a[c] : make_uint4(0u, 0u, 0u, 0u);
+        return;
+    }
     for (int c = threadIdx.x; c < D; c += blockDim.x)
         out[(size_t)r * D + c] = s >= 0 ? src[(size_t)s * D + c] : from_f32<T>(0.f);
 }
 
-extern "C" int aie_gather_rows(const void* src, const int* rows, void* out, int dtype, int n, int D, cudaStream_t st) {
+extern "C" int aie_gather_rows(const void* src, const int* rows, void* out, int dtype, int n, int D, int zero_fill,
+                               cudaStream_t st) {
     if (n <= 0) return 0;
     if (D <= 0) return AIE_BAD_ARG;
+    const size_t bytes = (size_t)D * (dtype == AIE_F32 ? 4 : 2);
+    const int vec = bytes % 16 == 0 && !(((size_t)src | (size_t)out) & 15);
+    const int threads = vec && bytes / 16 <= 128 ? 128 : 256;
     if (dtype == AIE_F32)
-        gather_rows_kernel<float><<<n, 256, 0, st>>>((const float*)src, rows, (float*)out, D);
+        launch_pdl(gather_rows_kernel<float>, dim3(n), dim3(threads), 0, st, (const float*)src, rows, (float*)out, D, zero_fill, vec);
     else if (dtype == AIE_BF16)
-        gather_rows_kernel<bf16><<<n, 256, 0, st>>>((const bf16*)src, rows, (bf16*)out, D);
+        launch_pdl(gather_rows_kernel<bf16>, dim3(n), dim3(threads), 0, st, (const bf16*)src, rows, (bf16*)out, D, zero_fill, vec);
     else
         return AIE_BAD_ARG;
     AIE_LAUNCH_CHECK();

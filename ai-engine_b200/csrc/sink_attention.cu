@@ -112,6 +112,8 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
                            const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
                            int e, int maps, int per_head, int write, unsigned* err) {
     extern __shared__ __align__(16) float np_sm[];     // q (H d) | k (G maps d) | 32
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x, tid = threadIdx.x;
     const int K = G * maps;                             // keys of a token
     const int nq = H * d, nk = K * d, nv = G * e;
@@ -205,6 +207,8 @@ head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
                            A* __restrict__ pages, const int* __restrict__ positions, const int* __restrict__ token_req,
                            const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
                            int e, int maps, int write, unsigned* err) {
+    pdl_launch_dependents();
+    pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int K = G * maps, nq = H * d, nk = K * d;
     const int hh = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);      // heads of q, then of k, then of v
@@ -256,9 +260,9 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
     if ((per_head || !q_w) && rot_dims == 0 && !mix_from && !v_keep && d <= 256 && e <= 256) {
         const dim3 grid(T, (H + G * maps + G + 7) / 8);
         if (dtype == AIE_F32)
-            head_normed_prepare_kernel<float><<<grid, 256, 0, stream>>>(proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+            launch_pdl(head_normed_prepare_kernel<float>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
         else if (dtype == AIE_BF16)
-            head_normed_prepare_kernel<bf16><<<grid, 256, 0, stream>>>(proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+            launch_pdl(head_normed_prepare_kernel<bf16>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
         else
             return AIE_BAD_ARG;
         AIE_LAUNCH_CHECK();
@@ -268,7 +272,7 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
 #define AIE_NAP(A)                                                                                                    \
     if (smem > 48 * 1024)                                                                                             \
         cudaFuncSetAttribute(normed_attn_prepare_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-    normed_attn_prepare_kernel<A><<<T, 256, smem, stream>>>(proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, halves, \
+    launch_pdl(normed_attn_prepare_kernel<A>, dim3(T), dim3(256), smem, stream, proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, halves, \
                                                            mix_from, lambda, v_keep, (A*)q_out, (A*)pages, positions, \
                                                            token_req, block_table, bt_width, num_pages, P, H, G, d, e, \
                                                            maps, per_head, write, err)

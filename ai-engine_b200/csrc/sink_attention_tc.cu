@@ -158,6 +158,8 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
     bf16* v_s = k_s + 2 * N * DK;                              // [2][64][DV]
     int* row_s = reinterpret_cast<int*>(v_s + 2 * N * DV);     // [2][64] cache rows of the tile's keys
 
+    pdl_launch_dependents();
+    pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int tile_i = (int)gridDim.y - 1 - (int)blockIdx.y;   // the list holds the tiles fewest keys first
     const int r = tiles[2 * tile_i], q_off = tiles[2 * tile_i + 1];
@@ -310,6 +312,8 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
     extern __shared__ __align__(128) unsigned char sd_smem[];
     __shared__ float mrg_m[SD_WARPS][SD_HEADS], mrg_l[SD_WARPS][SD_HEADS];
 
+    pdl_launch_dependents();
+    pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int s = blockIdx.x, di = blockIdx.z;
     const int group = H / G, gchunks = (group + GC - 1) / GC;
@@ -511,6 +515,8 @@ __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* 
                                  int S, float* __restrict__ out32) {
     __shared__ float w_s[SD_MAX_SPLITS];
     __shared__ float wsum_s;
+    pdl_launch_dependents();
+    pdl_wait();
     const int di = blockIdx.x, h = blockIdx.y;
     const int t = dec_tokens[di];
     const size_t base = ((size_t)di * H + h) * S;
@@ -567,7 +573,7 @@ extern "C" int aie_sink_attention_prefill(const void* q, const void* pages, void
         const size_t smem = (size_t)(SK_M * DK_ + 2 * 64 * DK_ + 2 * 64 * DV_) * sizeof(bf16) + 2 * 64 * sizeof(int);   \
         auto kern = sink_prefill_kernel<DK_, DV_>;                                                                    \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
-        kern<<<grid, SK_WARPS * 32, smem, stream>>>((const bf16*)q, (const bf16*)pages, (bf16*)out, gate, temp, slope, \
+        launch_pdl(kern, grid, dim3(SK_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)pages, (bf16*)out, gate, temp, slope, \
                                                     sink, tiles, q_start, q_len, ctx_len, block_table, bt_width,      \
                                                     num_pages, P, H, G, window, keep_first, chunk, maps, scale,       \
                                                     out32, err);                                                      \
@@ -598,7 +604,7 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
         const size_t smem = SdSmem<DK_, DV_>::bytes;                                                                  \
         auto kern = sink_decode_kernel<DK_, DV_>;                                                                     \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
-        kern<<<grid, SD_WARPS * 32, smem, stream>>>((const bf16*)q, (const bf16*)pages, (bf16*)out, part_o, part_lse, \
+        launch_pdl(kern, grid, dim3(SD_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)pages, (bf16*)out, part_o, part_lse, \
                                                     gate, temp, slope, sink, dec_tokens, positions, token_req,        \
                                                     block_table, bt_width, num_pages, P, H, G, GC, window,            \
                                                     keep_first, chunk, maps, scale, S, out32, err);                   \
@@ -610,7 +616,7 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
     if (S > 1) {
         const cudaError_t e1 = cudaGetLastError();
         if (e1 != cudaSuccess) return (int)e1;
-        sink_join_kernel<<<dim3(n, H), 128, 0, stream>>>(part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S, out32);
+        launch_pdl(sink_join_kernel, dim3(n, H), dim3(128), 0, stream, part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S, out32);
     }
     AIE_LAUNCH_CHECK();
 }

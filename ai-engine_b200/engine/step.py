@@ -12,6 +12,7 @@ Logits come back only for the rows that are wanted.
 """
 from __future__ import annotations
 
+import gc
 import os
 from dataclasses import dataclass
 from types import SimpleNamespace
@@ -264,8 +265,14 @@ class StepRunner:
             torch.cuda.synchronize()
             g = torch.cuda.CUDAGraph()
             n0 = LAUNCHES[0]
-            with torch.cuda.graph(g):
-                buf.graph_logits = self.model.forward(ctx, self.cache)
+            collecting = gc.isenabled()      # freeing an old engine's device objects inside a capture would spoil it
+            gc.disable()
+            try:
+                with torch.cuda.graph(g):
+                    buf.graph_logits = self.model.forward(ctx, self.cache)
+            finally:
+                if collecting:
+                    gc.enable()
             buf.graph_kernels = LAUNCHES[0] - n0
             buf.graph = g
             self.graphs_captured += 1

@@ -907,14 +907,14 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_t
     return out
 
 
-def gather_rows(src: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
-    """out[r] = src[rows[r]], zeros where rows[r] < 0."""
+def gather_rows(src: torch.Tensor, rows: torch.Tensor, zero_fill: bool = True) -> torch.Tensor:
+    """out[r] = src[rows[r]]; where rows[r] < 0, zeros, or nothing is written (zero_fill False)."""
     _dev(src, rows)
     out = torch.empty((rows.shape[0], src.shape[1]), dtype=src.dtype, device=src.device)
     lib = library("sequence_ops.cu")
     with region("gather_rows", 2 * _nb(out)):
         check(lib.aie_gather_rows(_p(src), _p(rows), _p(out), c_int(dtype_code(src)), c_int(rows.shape[0]),
-                                  c_int(src.shape[1]), _stream()), "gather_rows")
+                                  c_int(src.shape[1]), c_int(1 if zero_fill else 0), _stream()), "gather_rows")
     return out
 
 
@@ -922,13 +922,14 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, tile_w: torch.Tensor, out_d
                    err: torch.Tensor, row_src: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rows grouped in tiles of EXPERT_TILE, tile i multiplied with the weight w[tile_w[i]] of the stack w [E, N, K]
     (tile_w[i] < 0: the tile is skipped, its output rows are undefined).  x [rows, K], or, with `row_src`
-    [rows], the rows x[row_src[r]] (zeros for -1).  bfloat16 operands whose N is a multiple of 128 and K of 8
+    [rows], the rows x[row_src[r]] (where row_src[r] < 0 the output row is undefined: every row is a product of its
+    own).  bfloat16 operands whose N is a multiple of 128 and K of 8
     take the tcgen05 kernel, everything else the float32 kernel on the CUDA cores."""
     E, N, K = w.shape
     rows = tile_w.shape[0] * EXPERT_TILE
     out = torch.empty((rows, N), dtype=out_dtype, device=x.device)
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and N % 128 == 0 and K % 8 == 0:
-        xs = gather_rows(x, row_src) if row_src is not None else x
+        xs = gather_rows(x, row_src, zero_fill=False) if row_src is not None else x
         _dev(xs, w, tile_w, err)
         lib = library("gemm_tc.cu")
         with region("gemm_tc_grouped", _nb(xs, w, out), 2.0 * rows * N * K):
@@ -1064,9 +1065,18 @@ def scaled_sum(a: torch.Tensor, sa: float, b: torch.Tensor, sb: float) -> torch.
 PLAIN_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "relu_squared": 3}
 
 
-def activate(z: torch.Tensor, activation: str, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
-    """act(z) element by element (silu, relu, gelu_tanh, relu_squared), computed in float32."""
-    _dev(z)
+def activate(z: torch.Tensor, activation: str, out_dtype: Optional[torch.dtype] = None,
+             rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(z) element by element (silu, relu, gelu_tanh, relu_squared), computed in float32.  rows [n] int32, z [n, F]
+    float32: only the rows with rows[r] >= 0 (the others are undefined)."""
+    _dev(z, rows)
+    if rows is not None:
+        out = torch.empty(z.shape, dtype=out_dtype or z.dtype, device=z.device)
+        with region("activate", _nb(z, out)):
+            check(library("elementwise.cu").aie_activate_rows(
+                _p(z), c_int(dtype_code(z)), _p(rows), _p(out), c_int(dtype_code(out)), c_int(z.shape[0]), c_int(z.shape[1]),
+                c_int(PLAIN_ACTIVATIONS[activation]), _stream()), "activate_rows")
+        return out
     out = torch.empty(z.shape, dtype=out_dtype or z.dtype, device=z.device)
     lib = library("elementwise.cu")
     with region("activate", _nb(z, out)):

@@ -263,7 +263,7 @@ class GatedPostNormBlock(Block):
             raise ValueError("post-norm block: a gate without a feed-forward")
         self.gate, self.gate_bias = {}, {}
         self.joined = False            # the feed-forward's gate and its router are one weight
-        self.next_block = None
+        self.next_block, self.next_run = None, -1
 
     def tensor_specs(self):
         t = self.spec.tensors
@@ -288,8 +288,10 @@ class GatedPostNormBlock(Block):
     def flops(self, tokens, keys=0.0):
         return 2.0 * tokens * self.hidden * self.hidden * len(self.gated)
 
-    def set_next_block(self, block) -> None:
-        """The block that runs after this one in every step (only when every layer runs once)."""
+    def set_next_block(self, block, run: int) -> None:
+        """The block that runs after this one in every step, as entry `run` of the run order (only when every layer
+        runs once)."""
+        self.next_run = run
         self.next_block = block if isinstance(block, GatedPostNormBlock) and hasattr(block.p.get("shift"), "ahead") else None
 
     def forward(self, x, pending, ctx, caches):
@@ -330,9 +332,9 @@ class GatedPostNormBlock(Block):
         if not closes:
             return self.p[norm].add_normed(x, y, out_dtype=self.env.dtype, **options)
         nxt = self.next_block
-        if nxt is None or ctx.max_q_len != 1 or getattr(ctx, "step_cache", None) is None:
+        if nxt is None or ctx.max_q_len != 1:
             return self.p[norm].add_normed(x, y, **options)
-        cache = ctx.step_cache(nxt, "shift")
+        cache = ctx.cache.part_cache(self.next_run, "shift", ctx)
         h, shifted = self.p[norm].add_normed(x, y, out_dtype=self.env.dtype, next_shift=nxt.p["shift"].ahead(cache), ctx=ctx,
                                              **options)
         ctx.shifted_ahead = (nxt, h, shifted)

@@ -68,12 +68,12 @@ class Model:
         # every layer runs once is "the next block" the same at every run
         runs = [rs.layer for rs in self.order]
         if len(set(runs)) == len(runs):
-            for a, b in zip(runs, runs[1:]):
+            for i, (a, b) in enumerate(zip(runs, runs[1:])):
                 blk, nxt = self.layers[a].block, self.layers[b].block
                 if hasattr(blk, "set_next_norm") and hasattr(nxt, "first_norm"):
                     blk.set_next_norm(nxt.first_norm())
                 if hasattr(blk, "set_next_block"):
-                    blk.set_next_block(nxt)
+                    blk.set_next_block(nxt, i + 1)
         self.keeps_embedding_output = any(getattr(l.block, "needs_embedding_output", False) for l in self.layers)
         self.loaded = False
 
@@ -165,8 +165,7 @@ class Model:
         of the run order, for looking at a model layer by layer."""
         ctx.normed_ahead = None           # (norm, its output): made ahead by the block before the one that owns the norm
         ctx.shifted_ahead = None          # (block, stream, shifted stream): likewise, of the block that owns the shift
-        run_of = {id(self.layers[rs.layer].block): i for i, rs in enumerate(self.order)}
-        ctx.step_cache = lambda block, role: cache.part_cache(run_of[id(block)], role, ctx)
+        ctx.cache = cache
         x = self.embedding.forward(ctx)
         for pe in self.env.position_encodings.values():
             pe.add_to(x, ctx)

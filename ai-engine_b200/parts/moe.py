@@ -227,7 +227,7 @@ class RoutedMoE(FeedForward):
         if self.gated:
             act = ops.clamped_glu(gu, self.F, float("inf"), 1.0, 0.0, self.env.dtype)       # silu(gate) * up
         else:
-            act = ops.activate(gu, self.activation, self.env.dtype)
+            act = ops.activate(gu, self.activation, self.env.dtype, rows=row_token)
         y = ops.grouped_linear(act, self.w_down, tile_expert, torch.float32, ctx.err)
         if leave_rows and self.leaves_rows:
             return ops.ExpertRows(y, pair_row, weights)
