@@ -105,33 +105,36 @@ struct ShiftAhead {          // the next layer's token_shift (out null: not made
     int max_slots;
 };
 
-__device__ __forceinline__ float4 branch4(const BranchSource& b, int t, int c, int D) {
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (b.parts > 0) {
+// MODE 0: the parts of a product, gate or none;  1: one part each of branch and gate (a step of many tokens);
+// 2: expert rows.  Loads of what the previous kernel wrote; the gate's logits come back in g.
+template <int MODE>
+__device__ __forceinline__ void branch_loads(const BranchSource& b, int t, int c, int D, float4& v, float4& g) {
+    if (MODE == 1) {
+        v = load4<float>(b.y + (size_t)t * D + c);
+        g = load4<float>(b.z + (size_t)t * b.ldz + c);
+        return;
+    }
+    if (b.z) g = load4<float>(b.z + (size_t)t * b.ldz + c);
+    if (MODE == 0) {
         const float* p = b.y + (size_t)t * D + c;
         v = load4<float>(p);
 #pragma unroll 4
         for (int i = 1; i < b.parts; ++i) v = f4_add(v, load4<float>(p + i * b.stride));
-        if (b.bias) v = f4_add(v, load4<float>(b.bias + c));
     } else {
+        v = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
         for (int s = 0; s < b.top; ++s) {
             const int row = b.pair_row[(size_t)t * b.top + s];
-            if (row < 0) continue;
             const float w = b.weight[(size_t)t * b.top + s];
-            const float4 u = load4<float>(b.y + (size_t)row * D + c);
+            const float4 u = row >= 0 ? load4<float>(b.y + (size_t)row * D + c) : make_float4(0.f, 0.f, 0.f, 0.f);
             v = make_float4(fmaf(w, u.x, v.x), fmaf(w, u.y, v.y), fmaf(w, u.z, v.z), fmaf(w, u.w, v.w));
         }
     }
     if (b.z) {
         const float* p = b.z + (size_t)t * b.ldz + c;
-        float4 g = load4<float>(p);
 #pragma unroll 4
         for (int i = 1; i < b.zparts; ++i) g = f4_add(g, load4<float>(p + i * b.zstride));
-        if (b.zbias) g = f4_add(g, load4<float>(b.zbias + c));
-        v = make_float4(v.x * sigmoid_f(g.x), v.y * sigmoid_f(g.y), v.z * sigmoid_f(g.z), v.w * sigmoid_f(g.w));
     }
-    return v;
 }
 
 __device__ __forceinline__ float branch1(const BranchSource& b, int t, int c, int D) {
@@ -153,51 +156,80 @@ __device__ __forceinline__ float branch1(const BranchSource& b, int t, int c, in
     return v;
 }
 
-// One block per row; a thread owns NV float4 of it, blockDim float4 apart.
-template <int NV, typename O>
-__global__ void __launch_bounds__(NV == 1 ? 256 : 1024)
+// One block per row; a thread owns NV float4 of it, blockDim float4 apart.  What does not change between steps (norm
+// weight, biases, shift) is fetched before the wait for the previous kernel.
+template <int NV, int MODE, typename O>
+__global__ void __launch_bounds__(NV == 1 ? 1024 : 512)
 gated_norm_add_kernel(float* __restrict__ x, const BranchSource b, const float* __restrict__ w, O* __restrict__ out,
                       int D, float eps, const ShiftAhead sa, unsigned* err) {
     __shared__ float red[32];
     pdl_launch_dependents();
-    pdl_wait();
     const int t = blockIdx.x;
-    float4 v[NV], xv[NV];
+    float4 wv[NV], bv[NV], zb[NV];
+    if (NV == 1) {
+        const int c = threadIdx.x * 4;
+        wv[0] = bv[0] = zb[0] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < D) {
+            wv[0] = load4<float>(w + c);
+            if (b.bias) bv[0] = load4<float>(b.bias + c);
+            if (b.zbias) zb[0] = load4<float>(b.zbias + c);
+        }
+    }
+    pdl_wait();
+    float4 v[NV], g[NV], xv[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * 4;
+        v[k] = g[k] = xv[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c >= D) continue;
+        xv[k] = load4<float>(x + (size_t)t * D + c);
+        branch_loads<MODE>(b, t, c, D, v[k], g[k]);
+    }
+    int slot = -1;
+    if (sa.out) slot = sa.slots[sa.token_req[t]];
     float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int c = (threadIdx.x + k * blockDim.x) * 4;
-        v[k] = xv[k] = make_float4(0.f, 0.f, 0.f, 0.f);
         if (c >= D) continue;
-        xv[k] = load4<float>(x + (size_t)t * D + c);
-        v[k] = branch4(b, t, c, D);
+        if (NV > 1) {
+            if (b.bias) bv[k] = load4<float>(b.bias + c);
+            if (b.zbias) zb[k] = load4<float>(b.zbias + c);
+        }
+        if (b.bias) v[k] = f4_add(v[k], bv[k]);
+        if (b.z) {
+            if (b.zbias) g[k] = f4_add(g[k], zb[k]);
+            v[k] = make_float4(v[k].x * sigmoid_f(g[k].x), v[k].y * sigmoid_f(g[k].y), v[k].z * sigmoid_f(g[k].z),
+                               v[k].w * sigmoid_f(g[k].w));
+        }
         ss += v[k].x * v[k].x;
         ss += v[k].y * v[k].y;
         ss += v[k].z * v[k].z;
         ss += v[k].w * v[k].w;
     }
+    if (sa.out && (slot < 0 || slot >= sa.max_slots)) {
+        if (threadIdx.x == 0) atomicOr(err, AIE_DEV_SLOT_OOB);
+        slot = -1;
+    }
+    float4 old = make_float4(0.f, 0.f, 0.f, 0.f), sh = old;      // (with NV 1) the state and the shift, on their way meanwhile
+    if (NV == 1 && slot >= 0 && threadIdx.x * 4 < D) {
+        old = load4<float>(sa.state + (size_t)slot * D + threadIdx.x * 4);
+        sh = load4<float>(sa.shift + threadIdx.x * 4);
+    }
     ss = block_sum(ss, red);
     const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
-    int slot = -1;
-    if (sa.out) {
-        slot = sa.slots[sa.token_req[t]];
-        if (slot < 0 || slot >= sa.max_slots) {
-            if (threadIdx.x == 0) atomicOr(err, AIE_DEV_SLOT_OOB);
-            slot = -1;
-        }
-    }
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int c = (threadIdx.x + k * blockDim.x) * 4;
         if (c >= D) continue;
-        const float4 wv = load4<float>(w + c);
-        const float4 s = make_float4(xv[k].x + (v[k].x * rinv) * wv.x, xv[k].y + (v[k].y * rinv) * wv.y,
-                                     xv[k].z + (v[k].z * rinv) * wv.z, xv[k].w + (v[k].w * rinv) * wv.w);
+        if (NV > 1) wv[k] = load4<float>(w + c);
+        const float4 s = make_float4(xv[k].x + (v[k].x * rinv) * wv[k].x, xv[k].y + (v[k].y * rinv) * wv[k].y,
+                                     xv[k].z + (v[k].z * rinv) * wv[k].z, xv[k].w + (v[k].w * rinv) * wv[k].w);
         store4<float>(x + (size_t)t * D + c, s);
         if (out) store4<O>(out + (size_t)t * D + c, s);
         if (slot >= 0) {
             float* st = sa.state + (size_t)slot * D + c;
-            const float4 p = load4<float>(st), f = load4<float>(sa.shift + c);
+            const float4 p = NV == 1 ? old : load4<float>(st), f = NV == 1 ? sh : load4<float>(sa.shift + c);
             store4<O>((O*)sa.out + (size_t)t * D + c, make_float4(shifted_f(s.x, p.x, f.x), shifted_f(s.y, p.y, f.y),
                                                                   shifted_f(s.z, p.z, f.z), shifted_f(s.w, p.w, f.w)));
             store4<float>(st, s);
@@ -255,16 +287,23 @@ extern "C" int aie_gated_norm_add(float* x, const float* y, int parts, long long
                       (size_t)next_shift | (size_t)next_state | (size_t)next_out;
     const bool vec = D % 4 == 0 && ldz % 4 == 0 && stride % 4 == 0 && zstride % 4 == 0 && !(al & 15);
     const int f4 = D / 4;
-#define GO(NV, O)                                                                                                        \
-    launch_pdl(gated_norm_add_kernel<NV, O>, dim3(T), dim3(((f4 + NV - 1) / NV + 31) / 32 * 32), 0, st, x, b, w, (O*)out,  \
-               D, eps, sa, err)
+    const int mode = parts <= 0 ? 2 : (parts == 1 && zparts == 1 ? 1 : 0);
+    // few rows: a thread a float4, so that a row's latency is one load's; many: two and more, more blocks an SM
+    const int nv = f4 <= 256 || (T <= 2 * aie_sm_count() && f4 <= 1024) ? 1 : (f4 <= 1024 ? 2 : 4);
+#define GO(NV, M, O)                                                                                                     \
+    launch_pdl(gated_norm_add_kernel<NV, M, O>, dim3(T), dim3(((f4 + NV - 1) / NV + 31) / 32 * 32), 0, st, x, b, w,        \
+               (O*)out, D, eps, sa, err)
+#define GO_M(NV, O)                                                                                                      \
+    if (mode == 0) GO(NV, 0, O);                                                                                         \
+    else if (mode == 1) GO(NV, 1, O);                                                                                    \
+    else GO(NV, 2, O)
 #define GO_O(O)                                                                                                          \
-    if (vec && f4 <= 256) {                                                                                              \
-        GO(1, O);                                                                                                        \
+    if (vec && nv == 1) {                                                                                                \
+        GO_M(1, O);                                                                                                      \
+    } else if (vec && nv == 2) {                                                                                         \
+        GO_M(2, O);                                                                                                      \
     } else if (vec && f4 <= 2048) {                                                                                      \
-        GO(2, O);                                                                                                        \
-    } else if (vec && f4 <= 4096) {                                                                                      \
-        GO(4, O);                                                                                                        \
+        GO_M(4, O);                                                                                                      \
     } else {                                                                                                             \
         const size_t smem = (size_t)(D + 32) * sizeof(float);                                                            \
         if (smem > 200 * 1024) return AIE_UNSUPPORTED;                                                                   \
@@ -280,6 +319,7 @@ extern "C" int aie_gated_norm_add(float* x, const float* y, int parts, long long
         return AIE_BAD_ARG;
     }
 #undef GO_O
+#undef GO_M
 #undef GO
     AIE_LAUNCH_CHECK();
 }
@@ -287,24 +327,40 @@ extern "C" int aie_gated_norm_add(float* x, const float* y, int parts, long long
 // ---------------------------------------------------------------------------
 // out[t, c] = gelu_tanh(sum of the parts of z[t, c]) * table[ids[t], off + c]
 // ---------------------------------------------------------------------------
-template <typename E, typename O>
+__device__ __forceinline__ float gelu_tanh_f(float g) {
+    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+}
+
+// blockDim = (columns, rows of the block); VEC: four columns a thread
+template <typename E, typename O, bool VEC>
 __global__ void side_gate_kernel(const float* __restrict__ z, int parts, size_t stride, int ldz,
                                  const int* __restrict__ ids, const E* __restrict__ table, int vocab, int ld_table,
                                  int off, O* __restrict__ out, int T, int n, unsigned* err) {
     pdl_launch_dependents();
     pdl_wait();
-    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= (long long)T * n) return;
-    const int t = (int)(i / n), c = (int)(i % n);
+    const int t = blockIdx.x * blockDim.y + threadIdx.y;
+    if (t >= T) return;
     const int id = ids[t];
-    float g = 0.f;
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && threadIdx.x == 0) atomicOr(err, AIE_DEV_TOKEN_OOB);
+    const E* e = table + (size_t)(ok ? id : 0) * ld_table + off;
+    const float* p = z + (size_t)t * ldz;
+    if (VEC) {
+        for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+            float4 w = load4<E>(e + c), g = load4<float>(p + c);
+            if (!ok) w = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
-    for (int p = 0; p < parts; ++p) g += z[p * stride + (size_t)t * ldz + c];
-    float e = 0.f;
-    if (id >= 0 && id < vocab) e = to_f32<E>(table[(size_t)id * ld_table + off + c]);
-    else if (c == 0) atomicOr(err, AIE_DEV_TOKEN_OOB);
-    const float a = 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-    out[i] = from_f32<O>(a * e);
+            for (int i = 1; i < parts; ++i) g = f4_add(g, load4<float>(p + i * stride + c));
+            store4<O>(out + (size_t)t * n + c, make_float4(gelu_tanh_f(g.x) * w.x, gelu_tanh_f(g.y) * w.y,
+                                                           gelu_tanh_f(g.z) * w.z, gelu_tanh_f(g.w) * w.w));
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) {
+            float g = 0.f;
+            for (int i = 0; i < parts; ++i) g += p[i * stride + c];
+            out[(size_t)t * n + c] = from_f32<O>(ok ? gelu_tanh_f(g) * to_f32<E>(e[c]) : 0.f);
+        }
+    }
 }
 
 extern "C" int aie_side_gate(const float* z, int parts, long long stride, int ldz, const int* ids, const void* table,
@@ -312,16 +368,27 @@ extern "C" int aie_side_gate(const float* z, int parts, long long stride, int ld
                              unsigned* err, cudaStream_t st) {
     if (T <= 0) return 0;
     if (n <= 0 || parts < 1 || ldz < n || off < 0 || off + n > ld_table) return AIE_BAD_ARG;
-    const long long total = (long long)T * n;
-    const dim3 grid((unsigned)((total + 127) / 128));
+    const bool vec = n % 4 == 0 && ldz % 4 == 0 && stride % 4 == 0 && ld_table % 4 == 0 && off % 4 == 0 &&
+                     !(((size_t)z | (size_t)table | (size_t)out) & 15);
+    const int per = vec ? n / 4 : n;
+    const int bx = per >= 128 ? 128 : (per + 7) / 8 * 8, by = T >= 256 && bx <= 64 ? 128 / bx : 1;
+    const dim3 block(bx, by), grid((T + by - 1) / by);
 #define GO(E, O)                                                                                                      \
-    launch_pdl(side_gate_kernel<E, O>, grid, dim3(128), 0, st, z, parts, (size_t)stride, ldz, ids, (const E*)table,     \
-               vocab, ld_table, off, (O*)out, T, n, err)
-    if (table_dtype == AIE_F32 && out_dtype == AIE_F32) GO(float, float);
-    else if (table_dtype == AIE_BF16 && out_dtype == AIE_BF16) GO(bf16, bf16);
-    else if (table_dtype == AIE_F32 && out_dtype == AIE_BF16) GO(float, bf16);
-    else if (table_dtype == AIE_BF16 && out_dtype == AIE_F32) GO(bf16, float);
-    else return AIE_BAD_ARG;
+    if (vec) launch_pdl(side_gate_kernel<E, O, true>, grid, block, 0, st, z, parts, (size_t)stride, ldz, ids,           \
+                        (const E*)table, vocab, ld_table, off, (O*)out, T, n, err);                                     \
+    else launch_pdl(side_gate_kernel<E, O, false>, grid, block, 0, st, z, parts, (size_t)stride, ldz, ids,              \
+                    (const E*)table, vocab, ld_table, off, (O*)out, T, n, err)
+    if (table_dtype == AIE_F32 && out_dtype == AIE_F32) {
+        GO(float, float);
+    } else if (table_dtype == AIE_BF16 && out_dtype == AIE_BF16) {
+        GO(bf16, bf16);
+    } else if (table_dtype == AIE_F32 && out_dtype == AIE_BF16) {
+        GO(float, bf16);
+    } else if (table_dtype == AIE_BF16 && out_dtype == AIE_F32) {
+        GO(bf16, float);
+    } else {
+        return AIE_BAD_ARG;
+    }
 #undef GO
     AIE_LAUNCH_CHECK();
 }
@@ -415,7 +482,7 @@ __global__ void route_chosen_kernel(const float* __restrict__ z, int parts, size
         v[k] = s;
     }
     unsigned taken = 0u;                 // bit k: this lane's k-th logit is chosen
-    float best0 = 0.f, sum = 0.f;
+    float best0 = 0.f, sum = 0.f, mine = 0.f;      // lane l keeps the weight of choice l
     for (int s = 0; s < top; ++s) {
         float bv = -INFINITY;
         int be = 0x7fffffff;
@@ -440,14 +507,14 @@ __global__ void route_chosen_kernel(const float* __restrict__ z, int parts, size
         if (s == 0) best0 = bv;
         const float w = expf(bv - best0);
         sum += w;
-        if (lane == 0) {
-            ids[(size_t)t * top + s] = be;
-            weights[(size_t)t * top + s] = w;
+        if (lane == 0) ids[(size_t)t * top + s] = be;
+        if ((s & 31) == lane) {
+            if (s >= 32) weights[(size_t)t * top + s] = w;       // more than 32 choices: finished below
+            else mine = w;
         }
     }
-    __syncwarp();
-    if (lane == 0)
-        for (int s = 0; s < top; ++s) weights[(size_t)t * top + s] /= sum;
+    if (lane < top) weights[(size_t)t * top + lane] = mine / sum;
+    for (int s = lane + 32; s < top; s += 32) weights[(size_t)t * top + s] /= sum;
 }
 
 extern "C" int aie_route_chosen(const float* z, int parts, long long stride, int ldz, const float* bias, int T, int E,

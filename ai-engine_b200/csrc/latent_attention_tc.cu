@@ -13,14 +13,15 @@
 // in shared memory (eight threads a row); O += P V with the latent's columns split over the four warps, V being
 // the first `rank` columns of the same rows (ldmatrix.trans).  Few tokens in a step (decoding) cut each token's
 // chunks into `splits` parts that run as CTAs of their own and leave (maximum, sum, unnormalised output) for a
-// joining kernel.  A sink (exp(sink[h]) in the denominator, no key, no value) opens the running softmax of the first part.
+// joining kernel.  Weights enter the product with the rows rounded to bfloat16 and are summed so, or (PAIR) as two
+// bfloat16 terms each, 16 bits of mantissa, beside a float32 sum.  A sink (exp(sink[h]) in the denominator, no key, no value) opens the running softmax of the first part.
 #include "attention_prefill.cuh"
 
 #define LT_KEYS 64
 #define LT_ROWS 16
 #define LT_THREADS 128
 
-template <int CW, int TQ>      // latent columns per warp (rank = 4 CW); tokens per CTA
+template <int CW, int TQ, bool PAIR>      // latent columns per warp (rank = 4 CW); tokens per CTA; weights as two terms
 __global__ void __launch_bounds__(LT_THREADS * TQ)
 latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restrict__ pages, bf16* __restrict__ out,
                            float* __restrict__ part_o, float* __restrict__ part_ml, const int* __restrict__ tiles,
@@ -34,7 +35,8 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
     bf16* q_all = reinterpret_cast<bf16*>(lt_raw);                // [TQ][16][SK]
     bf16* k_s = q_all + TQ * LT_ROWS * SK;                        // [64][SK]
     bf16* p_all = k_s + LT_KEYS * SK;                             // [TQ][16][64 + 8]
-    float* s_all = reinterpret_cast<float*>(p_all + TQ * LT_ROWS * (LT_KEYS + 8));     // [TQ][16][64 + 1]
+    constexpr int PR = TQ * LT_ROWS * (LT_KEYS + 8);              // with PAIR a second plane: what rounding p left out
+    float* s_all = reinterpret_cast<float*>(p_all + (PAIR ? 2 : 1) * PR);              // [TQ][16][64 + 1]
     float* m_all = s_all + TQ * LT_ROWS * (LT_KEYS + 1);          // [TQ][16] running maximum
     float* l_all = m_all + TQ * LT_ROWS;                          // [TQ][16] running sum
     float* c_all = l_all + TQ * LT_ROWS;                          // [TQ][16] correction of this chunk
@@ -166,7 +168,8 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
                 const float p = (m_new == -INFINITY || v[i] == -INFINITY) ? 0.f : expf(v[i] - m_new);
                 const bf16 pb = __float2bfloat16_rn(p);
                 p_s[r * (LT_KEYS + 8) + g * 8 + i] = pb;
-                sum += __bfloat162float(pb);          // the sum of what the product will multiply
+                if (PAIR) p_s[PR + r * (LT_KEYS + 8) + g * 8 + i] = __float2bfloat16_rn(p - __bfloat162float(pb));
+                sum += PAIR ? p : __bfloat162float(pb);          // the sum of what the product will multiply
             }
 #pragma unroll
             for (int o = 4; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
@@ -193,6 +196,8 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
             for (int kk = 0; kk < LT_KEYS; kk += 16) {
                 unsigned a[4];
                 ldsm_x4(a[0], a[1], a[2], a[3], p_s + (lane & 15) * (LT_KEYS + 8) + kk + (lane >> 4) * 8);
+                unsigned a2[4];
+                if (PAIR) ldsm_x4(a2[0], a2[1], a2[2], a2[3], p_s + PR + (lane & 15) * (LT_KEYS + 8) + kk + (lane >> 4) * 8);
 #pragma unroll
                 for (int np = 0; np < NT / 2; ++np) {
                     unsigned b0, b1, b2, b3;
@@ -200,6 +205,10 @@ latent_attention_tc_kernel(const float* __restrict__ q_full, const bf16* __restr
                     ldsm_x4_t(b0, b1, b2, b3, k_s + (kk + (lane & 7) + ((lane >> 3) & 1) * 8) * SK + warp * CW + np * 16 + (lane >> 4) * 8);
                     mma16816(acc[2 * np], a, b0, b1);
                     mma16816(acc[2 * np + 1], a, b2, b3);
+                    if (PAIR) {
+                        mma16816(acc[2 * np], a2, b0, b1);
+                        mma16816(acc[2 * np + 1], a2, b2, b3);
+                    }
                 }
             }
         }
@@ -281,27 +290,29 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
                                        const int* tiles, int n_tiles, int tq, const int* q_start, const int* q_len,
                                        const int* ctx_len, const int* block_table, int bt_width,
                                        int num_pages, int P, int T, int H, int rank, int dk, int window, float scale,
-                                       int splits, const float* sink, unsigned* err, cudaStream_t st) {
+                                       int splits, const float* sink, int pair, unsigned* err, cudaStream_t st) {
     if (T <= 0 || n_tiles <= 0) return 0;
     if (rank < 64 || rank > 512 || rank % 64 || dk % 16 || dk < rank || dk > 1024 || H <= 0) return AIE_UNSUPPORTED;
     if (splits < 1 || splits > 64 || (splits > 1 && (!part_o || !part_ml)) || (tq != 1 && tq != 4)) return AIE_BAD_ARG;
     const int SK = dk + 8;
-    const size_t smem = (size_t)(tq * LT_ROWS + LT_KEYS) * SK * 2 + (size_t)tq * LT_ROWS * (LT_KEYS + 8) * 2 +
+    const size_t smem = (size_t)(tq * LT_ROWS + LT_KEYS) * SK * 2 + (size_t)tq * LT_ROWS * (LT_KEYS + 8) * 2 * (pair ? 2 : 1) +
                         (size_t)tq * (LT_ROWS * (LT_KEYS + 1) + 3 * LT_ROWS) * 4;
     if (smem > 220 * 1024) return AIE_UNSUPPORTED;
     dim3 grid(n_tiles, (H + LT_ROWS - 1) / LT_ROWS, splits);
     if (grid.y > 65535) return AIE_UNSUPPORTED;
-#define GO1(CWV, TQV)                                                                                                 \
+#define GO2(CWV, TQV, PV)                                                                                             \
     {                                                                                                                 \
-        auto kern = latent_attention_tc_kernel<CWV, TQV>;                                                             \
+        auto kern = latent_attention_tc_kernel<CWV, TQV, PV>;                                                         \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
         launch_pdl(kern, grid, dim3(LT_THREADS * TQV), smem, st, q_full, (const bf16*)pages, (bf16*)out, part_o, part_ml, tiles,    \
                                                    q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, H,   \
                                                    dk, window, scale, splits, sink, err);                                   \
     }
+#define GO1(CWV, TQV)                                                                                                 \
+    if (pair) GO2(CWV, TQV, true) else GO2(CWV, TQV, false)
 #define GO(CWV)                                                                                                       \
     case CWV:                                                                                                         \
-        if (tq == 1) GO1(CWV, 1) else GO1(CWV, 4)                                                                     \
+        if (tq == 1) { GO1(CWV, 1) } else { GO1(CWV, 4) }                                                             \
         break;
     switch (rank / 4) {
         GO(16) GO(32) GO(48) GO(64) GO(80) GO(96) GO(112) GO(128)
@@ -309,6 +320,7 @@ extern "C" int aie_latent_attention_tc(const float* q_full, const void* pages, v
     }
 #undef GO
 #undef GO1
+#undef GO2
     cudaError_t e = cudaGetLastError();
     if (e != cudaSuccess) return (int)e;
     if (splits > 1) launch_pdl(latent_join_kernel, dim3(T * H), dim3(128), 0, st, part_o, part_ml, (bf16*)out, splits, rank);

@@ -246,6 +246,67 @@ head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
     }
 }
 
+// The same for sizes in steps of 4 (d <= 128): groups of L lanes (a power of two, L >= d / 4) hold a head of q or k,
+// four elements a lane; the last blocks copy the values.
+template <typename A>
+__global__ void __launch_bounds__(256)
+head_normed_prepare4_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias,
+                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps, A* __restrict__ q_out,
+                            A* __restrict__ pages, const int* __restrict__ positions, const int* __restrict__ token_req,
+                            const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
+                            int e, int maps, int L, int head_blocks, int write, unsigned* err) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, lane = threadIdx.x & 31;
+    const int K = G * maps, nq = H * d, nk = K * d, w_row = maps * d + e;
+    const float* row = proj + (size_t)t * ld;
+    A* base = nullptr;                                   // the token's place in the page, of key/value head 0
+    const bool values = blockIdx.y >= head_blocks;
+    const int per = 32 / L;
+    const int hh = (blockIdx.y * 8 + (threadIdx.x >> 5)) * per + lane / L, c = (lane & (L - 1)) * 4;
+    if (values || hh >= H) {
+        const int pos = positions[t], pidx = pos / P;
+        const int page = (pos >= 0 && pidx < bt_width) ? block_table[(size_t)token_req[t] * bt_width + pidx] : -1;
+        if (page >= 0 && page < num_pages) base = pages + ((size_t)page * G * P + (pos - pidx * P)) * w_row;
+        else if (write && (threadIdx.x & 31) == 0) atomicOr(err, AIE_DEV_PAGE_OOB);
+    }
+    if (values) {
+        const int i = ((blockIdx.y - head_blocks) * blockDim.x + threadIdx.x) * 4;
+        if (i >= G * e || !base || !write) return;
+        float4 v = load4<float>(row + nq + nk + i);
+        if (bias) {
+            const float4 b = load4<float>(bias + nq + nk + i);
+            v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+        }
+        const int g = i / e;
+        store4<A>(base + (size_t)g * P * w_row + maps * d + (i - g * e), v);
+        return;
+    }
+    const bool on = hh < H + K && c < d;
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), w = x;
+    if (on) {
+        x = load4<float>(row + hh * d + c);
+        if (bias) {
+            const float4 b = load4<float>(bias + hh * d + c);
+            x = make_float4(x.x + b.x, x.y + b.y, x.z + b.z, x.w + b.w);
+        }
+        if (q_w) w = load4<float>((hh < H ? q_w : k_w) + c);
+    }
+    if (q_w) {
+        float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        for (int o = L >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+        x = make_float4((x.x * inv) * w.x, (x.y * inv) * w.y, (x.z * inv) * w.z, (x.w * inv) * w.w);
+    }
+    if (!on) return;
+    if (hh < H) {
+        store4<A>(q_out + (size_t)t * nq + hh * d + c, x);
+    } else if (base && write) {
+        const int k = hh - H;
+        store4<A>(base + (size_t)(k / maps) * P * w_row + (k % maps) * d + c, x);
+    }
+}
+
 extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* bias, const float* q_w, const float* k_w,
                                        float eps, const float* inv_freq, int rot_dims, int halves, const float* mix_from,
                                        const float* lambda, float* v_keep, void* q_out, void* pages, int dtype,
@@ -258,6 +319,18 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
         (mix_from && !lambda) || (q_w && !k_w) || (rot_dims > 0 && !inv_freq))
         return AIE_BAD_ARG;
     if ((per_head || !q_w) && rot_dims == 0 && !mix_from && !v_keep && d <= 256 && e <= 256) {
+        const size_t al = (size_t)proj | (size_t)bias | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)pages;
+        if (d % 4 == 0 && e % 4 == 0 && ld % 4 == 0 && d <= 128 && !(al & 15) && (dtype == AIE_F32 || dtype == AIE_BF16)) {
+            int L = 1;
+            while (L * 4 < d) L *= 2;
+            const int hb = (H + G * maps + 8 * (32 / L) - 1) / (8 * (32 / L)), vb = (G * e / 4 + 255) / 256;
+            const dim3 grid4(T, hb + vb);
+            if (dtype == AIE_F32)
+                launch_pdl(head_normed_prepare4_kernel<float>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, write, err);
+            else
+                launch_pdl(head_normed_prepare4_kernel<bf16>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, write, err);
+            AIE_LAUNCH_CHECK();
+        }
         const dim3 grid(T, (H + G * maps + G + 7) / 8);
         if (dtype == AIE_F32)
             launch_pdl(head_normed_prepare_kernel<float>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);

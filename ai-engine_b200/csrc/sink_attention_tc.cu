@@ -539,6 +539,7 @@ __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* 
     for (int e = threadIdx.x; e < DV; e += blockDim.x) {
         const float* src = part_o + base * DV + e;
         float A = 0.f;
+#pragma unroll 8
         for (int s = 0; s < S; ++s) A += w_s[s] * src[(size_t)s * DV];
         const size_t at = ((size_t)t * H + h) * DV + e;
         if (out32) out32[at] = A * inv;

@@ -790,12 +790,13 @@ def latent_prepare(proj: torch.Tensor, H: int, d: int, rot: int, rank: int, c_we
 
 def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table: torch.Tensor, rank: int,
                      scale: float, window: int, out_dtype: torch.dtype, work=None,
-                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     sink: Optional[torch.Tensor] = None, exact_weights: bool = False) -> torch.Tensor:
     """softmax over the visible cache rows of (q_full . row) * scale, times the rows' first `rank` elements:
     [T, H, rank].  q_full [T, H, dk] float32; pages [num_pages, 1, P, dk].  `work`: the step's units of tokens
     (`tiles` [n, 2], `tq`) for the tensor-core kernel, which bfloat16 takes when the sizes fit (a latent of
     64 .. 512 in steps of 64, rows a multiple of 16); everything else takes the plain kernel.  sink [H] float32: the
-    denominator also holds exp(sink[h])."""
+    denominator also holds exp(sink[h]).  exact_weights: the tensor-core kernel multiplies weights of 16 bits of mantissa
+    (two terms) instead of 8."""
     _dev(q_full, pages, block_table, sink)
     T, H, dk = q_full.shape
     if (q_full.dtype != torch.float32 or pages.shape[3] != dk or pages.shape[1] != 1
@@ -812,7 +813,7 @@ def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table
         cost = (cost[0] + rows * dk * pages.element_size(), 2.0 * pairs * H * (dk + rank))
     if (work is not None and pages.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and rank % 64 == 0
             and 64 <= rank <= 512 and dk % 16 == 0 and dk <= 1024
-            and (work.tq * 16 + 64) * (dk + 8) * 2 + work.tq * 7000 <= 220 * 1024):
+            and (work.tq * 16 + 64) * (dk + 8) * 2 + work.tq * (9400 if exact_weights else 7000) <= 220 * 1024):
         # tensor cores; a step of few tokens cuts each token's keys into parts so that the grid fills the machine
         keys = ctx.bt_width * ctx.page_size if ctx.bucketed else ctx.max_total_len
         if window > 0:
@@ -830,7 +831,7 @@ def latent_attention(q_full: torch.Tensor, pages: torch.Tensor, ctx, block_table
                                               _p(ctx.q_len), _p(ctx.ctx_len), _p(block_table), c_int(block_table.shape[1]),
                                               c_int(pages.shape[0]), c_int(pages.shape[2]), c_int(T), c_int(H),
                                               c_int(rank), c_int(dk), c_int(window), c_float(scale), c_int(splits),
-                                              _p(sink), _p(ctx.err), _stream()), "latent_attention_tc")
+                                              _p(sink), c_int(1 if exact_weights else 0), _p(ctx.err), _stream()), "latent_attention_tc")
         return out
     lib = library("latent_attention.cu")
     with region("latent_attention", *cost):
@@ -907,19 +908,20 @@ def linear_recurrence(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay_t
     return out
 
 
-def gather_rows(src: torch.Tensor, rows: torch.Tensor, zero_fill: bool = True) -> torch.Tensor:
-    """out[r] = src[rows[r]]; where rows[r] < 0, zeros, or nothing is written (zero_fill False)."""
+def gather_rows(src: torch.Tensor, rows: torch.Tensor, zero_fill: bool = True, live: Optional[int] = None) -> torch.Tensor:
+    """out[r] = src[rows[r]]; where rows[r] < 0, zeros, or nothing is written (zero_fill False).  live: how many rows
+    are not padding (for the byte count of a profile)."""
     _dev(src, rows)
     out = torch.empty((rows.shape[0], src.shape[1]), dtype=src.dtype, device=src.device)
     lib = library("sequence_ops.cu")
-    with region("gather_rows", 2 * _nb(out)):
+    with region("gather_rows", 2 * (live if live is not None and not zero_fill else out.shape[0]) * out.shape[1] * out.element_size()):
         check(lib.aie_gather_rows(_p(src), _p(rows), _p(out), c_int(dtype_code(src)), c_int(rows.shape[0]),
                                   c_int(src.shape[1]), c_int(1 if zero_fill else 0), _stream()), "gather_rows")
     return out
 
 
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, tile_w: torch.Tensor, out_dtype: torch.dtype,
-                   err: torch.Tensor, row_src: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   err: torch.Tensor, row_src: Optional[torch.Tensor] = None, live: Optional[int] = None) -> torch.Tensor:
     """Rows grouped in tiles of EXPERT_TILE, tile i multiplied with the weight w[tile_w[i]] of the stack w [E, N, K]
     (tile_w[i] < 0: the tile is skipped, its output rows are undefined).  x [rows, K], or, with `row_src`
     [rows], the rows x[row_src[r]] (where row_src[r] < 0 the output row is undefined: every row is a product of its
@@ -929,7 +931,7 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, tile_w: torch.Tensor, out_d
     rows = tile_w.shape[0] * EXPERT_TILE
     out = torch.empty((rows, N), dtype=out_dtype, device=x.device)
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and N % 128 == 0 and K % 8 == 0:
-        xs = gather_rows(x, row_src, zero_fill=False) if row_src is not None else x
+        xs = gather_rows(x, row_src, zero_fill=False, live=live) if row_src is not None else x
         _dev(xs, w, tile_w, err)
         lib = library("gemm_tc.cu")
         with region("gemm_tc_grouped", _nb(xs, w, out), 2.0 * rows * N * K):
@@ -1066,13 +1068,13 @@ PLAIN_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "relu_squared": 3}
 
 
 def activate(z: torch.Tensor, activation: str, out_dtype: Optional[torch.dtype] = None,
-             rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+             rows: Optional[torch.Tensor] = None, live: Optional[int] = None) -> torch.Tensor:
     """act(z) element by element (silu, relu, gelu_tanh, relu_squared), computed in float32.  rows [n] int32, z [n, F]
-    float32: only the rows with rows[r] >= 0 (the others are undefined)."""
+    float32: only the rows with rows[r] >= 0 (the others are undefined), `live` of them (for the byte count of a profile)."""
     _dev(z, rows)
     if rows is not None:
         out = torch.empty(z.shape, dtype=out_dtype or z.dtype, device=z.device)
-        with region("activate", _nb(z, out)):
+        with region("activate", (live if live is not None else z.shape[0]) * z.shape[1] * (z.element_size() + out.element_size())):
             check(library("elementwise.cu").aie_activate_rows(
                 _p(z), c_int(dtype_code(z)), _p(rows), _p(out), c_int(dtype_code(out)), c_int(z.shape[0]), c_int(z.shape[1]),
                 c_int(PLAIN_ACTIVATIONS[activation]), _stream()), "activate_rows")

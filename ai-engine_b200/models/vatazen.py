@@ -37,7 +37,7 @@ def build_vatazen_spec(cfg: VatazenConfig) -> ModelSpec:
         if l.type == "latent_attention":
             parts["mixer"] = PartSpec("latent_attention", dict(
                 hidden_size=D, num_heads=m.heads, head_dim=m.dim, rot_dim=m.rot_dim, value_dim=m.vdim, kv_rank=m.kv_rank,
-                scale=m.scale, window=m.mask_size, eps=eps, sink=True, position_encoding=_rotary(encodings, m)),
+                scale=m.scale, window=m.mask_size, eps=eps, sink=True, exact_weights=True, position_encoding=_rotary(encodings, m)),
                 dict(q=q + "q", dkv=q + "dkv", dkv_norm=q + "dkv.norm", uk=q + "uk", uv=q + "uv", sink=q + "sink", o=q + "o"))
         else:
             parts["mixer"] = PartSpec("differential_attention", dict(

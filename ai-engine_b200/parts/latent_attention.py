@@ -49,7 +49,8 @@ class LatentAttention(Mixer):
     """params: hidden_size, num_heads, head_dim (unrotated part), rot_dim, value_dim, kv_rank, scale, window
     (0 = all keys), cache_window (the window the cached rows must outlive: the widest of all layers that read
     them; default = window), eps (of the latents' norms), position_encoding (name of a rotary encoding over rot_dim
-    or fewer elements, either layout), shares_cache, q_rank (0: the queries are projected directly), head_gate, sink (default False).
+    or fewer elements, either layout), shares_cache, q_rank (0: the queries are projected directly), head_gate, sink (default False),
+    exact_weights (default False: the tensor-core kernel rounds softmax weights to bfloat16).
     tensors: q [H (d + rot), hidden] (or, with q_rank: dq [q_rank, hidden], dq_norm [q_rank], uq [H (d + rot),
     q_rank]), dkv [kv_rank + rot, hidden], dkv_norm [kv_rank], uk [H d, kv_rank], uv [H dv, kv_rank], o [hidden,
     H dv], g [H, hidden], sink [H]."""
@@ -72,7 +73,7 @@ class LatentAttention(Mixer):
             raise ValueError("latent attention: the rotation is wider than rot_dim")
         self.halves = self.rope is not None and not getattr(self.rope, "interleaved", False)
         self.q_rank, self.head_gate = int(p.get("q_rank") or 0), bool(p.get("head_gate"))
-        self.has_sink = bool(p.get("sink"))
+        self.has_sink, self.exact_weights = bool(p.get("sink")), bool(p.get("exact_weights"))
         self.magnitude = float(getattr(self.rope, "magnitude", 1.0)) if self.rope is not None else 1.0
         if (self.q_rank or self.head_gate) and self.shares_cache:
             raise ValueError("latent attention: a layer that reads another's cache has neither a query latent nor a gate")
@@ -159,7 +160,8 @@ class LatentAttention(Mixer):
                                              magnitude=self.magnitude)
         ops.head_linear(q_plain, self.w_ukT, q_full)
         mixed = ops.latent_attention(q_full, cache.k_pages, ctx, cache.block_table, self.rank, self.scale,
-                                     self.window, self.env.dtype, ctx.plan(LATENT_WORK), sink=self.sink)
+                                     self.window, self.env.dtype, ctx.plan(LATENT_WORK), sink=self.sink,
+                                     exact_weights=self.exact_weights)
         a = torch.empty((T, self.H, self.dv), dtype=self.env.dtype, device=h.device)
         ops.head_linear(mixed, self.w_uv, a)
         a = a.view(T, self.H * self.dv)

@@ -79,7 +79,7 @@ class TableMoE(FeedForward):
     def forward(self, h, ctx):
         T, D, F = h.shape[0], self.hidden, self.F
         row_token, pair_row, tile_expert = ops.expert_plan(ctx.token_ids, self.table, self.E, ctx.err)
-        gu = ops.grouped_linear(h, self.w_gu, tile_expert, torch.float32, ctx.err, row_src=row_token)
+        gu = ops.grouped_linear(h, self.w_gu, tile_expert, torch.float32, ctx.err, row_src=row_token, live=pair_row.numel())
         act = ops.clamped_glu(gu, F, self.limit, self.alpha, self.shift, self.env.dtype)
         y = ops.grouped_linear(act, self.w_down, tile_expert, torch.float32, ctx.err)
         shared = gate = None
@@ -223,11 +223,11 @@ class RoutedMoE(FeedForward):
             pair_row = torch.full((ids.numel(),), -2, dtype=torch.int32, device=h.device)
             return ops.expert_combine_weighted(y, pair_row, weights, h, shared)
         row_token, pair_row, tile_expert = ops.expert_plan(None, ids, self.E, ctx.err, identity=self.ident)
-        gu = ops.grouped_linear(h, self.w_gu, tile_expert, torch.float32, ctx.err, row_src=row_token)
+        gu = ops.grouped_linear(h, self.w_gu, tile_expert, torch.float32, ctx.err, row_src=row_token, live=pair_row.numel())
         if self.gated:
             act = ops.clamped_glu(gu, self.F, float("inf"), 1.0, 0.0, self.env.dtype)       # silu(gate) * up
         else:
-            act = ops.activate(gu, self.activation, self.env.dtype, rows=row_token)
+            act = ops.activate(gu, self.activation, self.env.dtype, rows=row_token, live=ids.numel())
         y = ops.grouped_linear(act, self.w_down, tile_expert, torch.float32, ctx.err)
         if leave_rows and self.leaves_rows:
             return ops.ExpertRows(y, pair_row, weights)

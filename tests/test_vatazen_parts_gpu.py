@@ -143,7 +143,7 @@ def test_side_input(dtype, D, n, levels, T):
     assert int(ctx.err.item()) == 1
 
 
-@pytest.mark.parametrize("E,top", [(8, 3), (1, 1), (5, 5), (33, 4), (64, 8), (100, 7), (250, 2), (700, 9)])
+@pytest.mark.parametrize("E,top", [(8, 3), (1, 1), (5, 5), (33, 4), (64, 8), (100, 7), (250, 2), (700, 9), (90, 70)])
 def test_router_choices_and_weights(E, top):
     from ai_engine_b200.kernels import ops
     gen = torch.Generator().manual_seed(E)
@@ -224,7 +224,7 @@ def test_difference_of_two_maps(dtype, H, e):
 
 
 # ---------------------------------------------------------------------------------------------------
-def latent_part(m, hidden, eps, dtype, gen, tie_keys=False):
+def latent_part(m, hidden, eps, dtype, gen, tie_keys=False, exact=True):
     from ai_engine_b200.parts import LatentAttention, PartSpec, RotaryEncoding
     H, d, r, e, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     t = {"q": rnd(gen, H * (d + r), hidden, std=0.3), "dkv": rnd(gen, rank + r, hidden, std=0.3),
@@ -246,7 +246,7 @@ def latent_part(m, hidden, eps, dtype, gen, tie_keys=False):
         pe = "r"
     spec = PartSpec("latent_attention", dict(
         hidden_size=hidden, num_heads=H, head_dim=d, rot_dim=r, value_dim=e, kv_rank=rank, scale=m["scale"],
-        window=(m.get("mask") or {}).get("size", 0), eps=eps, sink=True, position_encoding=pe),
+        window=(m.get("mask") or {}).get("size", 0), eps=eps, sink=True, exact_weights=exact, position_encoding=pe),
         dict(q="q", dkv="dkv", dkv_norm="dkv.norm", uk="uk", uv="uv", sink="sink", o="o"))
     return load(LatentAttention(spec, e_), t, DT[dtype]), t
 
