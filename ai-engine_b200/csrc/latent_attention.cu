@@ -13,7 +13,7 @@
 //   of their own (`kv`, rows ld_kv floats apart) when the queries are made by a second product.
 // latent_attention: one block per (token, head); keys in chunks of 128 that start at multiples of 128 of the
 //   absolute key position with a running maximum and sum, so a row's additions depend on its position only.
-//   `sink` (a number per head, or null): the denominator also holds exp(sink[h]), which has no key and no value.
+//   `sink` (a number per head, or null): exp(sink[h]) joins the denominator and adds nothing to the output.
 #include "common.cuh"
 
 #define LAT_CHUNK 128

@@ -14,7 +14,7 @@
 // the first `rank` columns of the same rows (ldmatrix.trans).  Few tokens in a step (decoding) cut each token's
 // chunks into `splits` parts that run as CTAs of their own and leave (maximum, sum, unnormalised output) for a
 // joining kernel.  Weights enter the product with the rows rounded to bfloat16 and are summed so, or (PAIR) as two
-// bfloat16 terms each, 16 bits of mantissa, beside a float32 sum.  A sink (exp(sink[h]) in the denominator, no key, no value) opens the running softmax of the first part.
+// bfloat16 terms each, 16 bits of mantissa, beside a float32 sum.  A sink (exp(sink[h]) in the denominator, nothing in the output) opens the running softmax of the first part.
 #include "attention_prefill.cuh"
 
 #define LT_KEYS 64

@@ -13,8 +13,8 @@ one key/value head for all query heads, for prompts and decoded tokens alike.
 The queries may go through a latent of their own (`q_rank`): c_q = RMSnorm(W_dq h) with a weight, q = W_uq c_q.  A
 gate per head (`head_gate`) multiplies head h's output by sigmoid(W_g h)_h; it is applied to the head's values before
 the output projection.  The rotation pairs neighbours or halves, as its encoding says, and carries its encoding's
-magnitude.  A softmax may leak into a sink (`sink`): its denominator also holds exp(sink_h), a learned number per head
-that has no key and no value and is not scaled.
+magnitude.  A softmax may leak into a sink (`sink`): exp(sink_h) joins its denominator, one learned score per
+head with nothing behind it, taken as it is.
 
 A layer may read another layer's cache (`shares_cache`): it has no latent projection of its own and writes
 nothing; the run order names the layer whose rows it reads.
