@@ -21,3 +21,6 @@ __all__.append("FokisunConfig")
 from .vatazen import VatazenConfig  # noqa: E402
 
 __all__.append("VatazenConfig")
+from .kagatar import KagatarConfig  # noqa: E402
+
+__all__.append("KagatarConfig")

@@ -271,11 +271,160 @@ extern "C" int aie_add_rmsnorm(float* x, const void* delta, int delta_dtype, con
 }
 
 // ---------------------------------------------------------------------------
+// Two RMS norms of one row that differ in their weights only, ahead of two branches that read the same stream:
+//   s = x[t] (+ the sum of `parts` deltas) (+ extra[t]) (+ step);  x[t] = s where anything was added;
+//   out1[t] = s / sqrt(mean(s^2) + eps) * w1,   out2[t] the same with w2 (null: no second output).
+// extra is a second stream, step one row for all tokens (both optional).  V float4 a thread and D == 4 V blockDim, or
+// V == 0: any D, the row in shared memory.
+// ---------------------------------------------------------------------------
+__device__ __forceinline__ float4 add4(float4 a, float4 b) {
+    return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w);
+}
+
+template <int V, typename W, typename O>
+__global__ void __launch_bounds__(1024)
+add_rmsnorm_pair_kernel(float* __restrict__ x, const float* __restrict__ delta, int parts, size_t part_stride,
+                        const float* __restrict__ extra, const float* __restrict__ step, const W* __restrict__ w1,
+                        const W* __restrict__ w2, O* __restrict__ out1, O* __restrict__ out2, int D, float eps) {
+    __shared__ float red[32];
+    const size_t at = (size_t)blockIdx.x * D;
+    const int i = threadIdx.x, nt = blockDim.x;
+    float4 g1[V], g2[V], st[V];
+    const bool on = V > 1 || i < D / 4;
+    if (V == 1 && on) {                          // few rows: the constants are on their way before the wait
+        g1[0] = load4<W>(w1 + 4 * i);
+        if (w2) g2[0] = load4<W>(w2 + 4 * i);
+        if (step) st[0] = load4<float>(step + 4 * i);
+    }
+    pdl_launch_dependents();
+    pdl_wait();
+    float4 s[V];
+    float ss = 0.f;
+    if (on) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) s[k] = reinterpret_cast<const float4*>(x + at)[i + k * nt];
+        int p = 0;
+        for (; V == 1 && p + 4 <= parts; p += 4) {           // four loads in flight, added in order
+            float4 dl[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) dl[u] = load4<float>(delta + (size_t)(p + u) * part_stride + at + 4 * i);
+#pragma unroll
+            for (int u = 0; u < 4; ++u) s[0] = add4(s[0], dl[u]);
+        }
+        for (; p < parts; ++p)
+#pragma unroll
+            for (int k = 0; k < V; ++k) s[k] = add4(s[k], load4<float>(delta + (size_t)p * part_stride + at + 4 * (i + k * nt)));
+        if (extra) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) s[k] = add4(s[k], load4<float>(extra + at + 4 * (i + k * nt)));
+        }
+        if (step) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) s[k] = add4(s[k], V == 1 ? st[k] : load4<float>(step + 4 * (i + k * nt)));
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+            ss += s[k].x * s[k].x;
+            ss += s[k].y * s[k].y;
+            ss += s[k].z * s[k].z;
+            ss += s[k].w * s[k].w;
+        }
+    }
+    ss = block_sum(ss, red);
+    const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+    if (!on) return;
+    const bool stored = parts > 0 || extra || step;
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+        const int c = 4 * (i + k * nt);
+        if (stored) *reinterpret_cast<float4*>(x + at + c) = s[k];
+        const float4 n = make_float4(s[k].x * rinv, s[k].y * rinv, s[k].z * rinv, s[k].w * rinv);
+        if (V > 1) g1[k] = load4<W>(w1 + c);
+        store4<O>(out1 + at + c, make_float4(n.x * g1[k].x, n.y * g1[k].y, n.z * g1[k].z, n.w * g1[k].w));
+        if (w2) {
+            if (V > 1) g2[k] = load4<W>(w2 + c);
+            store4<O>(out2 + at + c, make_float4(n.x * g2[k].x, n.y * g2[k].y, n.z * g2[k].z, n.w * g2[k].w));
+        }
+    }
+}
+
+template <typename W, typename O>
+__global__ void __launch_bounds__(512)
+add_rmsnorm_pair_any_kernel(float* __restrict__ x, const float* __restrict__ delta, int parts, size_t part_stride,
+                            const float* __restrict__ extra, const float* __restrict__ step, const W* __restrict__ w1,
+                            const W* __restrict__ w2, O* __restrict__ out1, O* __restrict__ out2, int D, float eps) {
+    extern __shared__ float srow[];   // D floats + 32
+    float* red = srow + D;
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t at = (size_t)blockIdx.x * D;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        float s = x[at + i];
+        for (int p = 0; p < parts; ++p) s += delta[p * part_stride + at + i];
+        if (extra) s += extra[at + i];
+        if (step) s += step[i];
+        srow[i] = s;
+        ss += s * s;
+    }
+    ss = block_sum(ss, red);
+    const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+    const bool stored = parts > 0 || extra || step;
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        const float s = srow[i];
+        if (stored) x[at + i] = s;
+        out1[at + i] = from_f32<O>((s * rinv) * to_f32<W>(w1[i]));
+        if (w2) out2[at + i] = from_f32<O>((s * rinv) * to_f32<W>(w2[i]));
+    }
+}
+
+template <typename W, typename O>
+static int launch_rmsnorm_pair(float* x, const float* delta, int parts, size_t stride, const float* extra, const float* step,
+                               const void* w1, const void* w2, void* out1, void* out2, int T, int D, float eps,
+                               cudaStream_t st) {
+    const size_t al = (size_t)x | (size_t)delta | (size_t)extra | (size_t)step | (size_t)w1 | (size_t)w2 | (size_t)out1 | (size_t)out2;
+    const bool vec = !(al & 15) && D % 4 == 0 && (parts == 0 || stride % 4 == 0);
+#define AIE_RP(KERN, THREADS, SMEM)                                                                                        \
+    launch_pdl(KERN, dim3(T), dim3(THREADS), SMEM, st, x, delta, parts, stride, extra, step, (const W*)w1, (const W*)w2, (O*)out1, (O*)out2, D, eps)
+    if (vec && T >= 256 && D % 512 == 0 && D <= 16384) {
+        AIE_RP((add_rmsnorm_pair_kernel<4, W, O>), D / 16, 0);
+    } else if (vec && D <= 4096) {
+        AIE_RP((add_rmsnorm_pair_kernel<1, W, O>), ((D / 4) + 31) / 32 * 32, 0);
+    } else {
+        const size_t smem = (size_t)(D + 32) * sizeof(float);
+        if (smem > 200 * 1024) return AIE_UNSUPPORTED;
+        auto k = add_rmsnorm_pair_any_kernel<W, O>;
+        if (smem > 48 * 1024) cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        AIE_RP(k, D >= 1024 ? 512 : 256, smem);
+    }
+#undef AIE_RP
+    AIE_LAUNCH_CHECK();
+}
+
+extern "C" int aie_add_rmsnorm_pair(float* x, const float* delta, int parts, long long part_stride, const float* extra,
+                                    const float* step, const void* w1, const void* w2, int w_dtype, void* out1, void* out2,
+                                    int out_dtype, int T, int D, float eps, cudaStream_t st) {
+    if (T <= 0) return 0;
+    if (D <= 0 || parts < 0 || (parts > 0 && !delta) || !w1 || !out1 || (w2 && !out2)) return AIE_BAD_ARG;
+#define GO(W, O) return launch_rmsnorm_pair<W, O>(x, delta, parts, (size_t)part_stride, extra, step, w1, w2, out1, out2, T, D, eps, st)
+    if (w_dtype == AIE_F32 && out_dtype == AIE_F32) GO(float, float);
+    if (w_dtype == AIE_F32 && out_dtype == AIE_BF16) GO(float, bf16);
+    if (w_dtype == AIE_BF16 && out_dtype == AIE_F32) GO(bf16, float);
+    if (w_dtype == AIE_BF16 && out_dtype == AIE_BF16) GO(bf16, bf16);
+#undef GO
+    return AIE_BAD_ARG;
+}
+
+// ---------------------------------------------------------------------------
 // a[t, f] = silu(gate) * up   (crates/ai-engine-runtime/src/arch/ffn.rs:50-54), silu(z) = z * sigmoid(z)
 // in float32.  block == 0: gu[t] = [gate (F) | up (F)].  block > 0: gu[t] is in groups of
 // 2 * block columns, `block` gate columns followed by their `block` up columns.
 // ---------------------------------------------------------------------------
-// the activation of a gated unit: 0 silu, 1 relu, 2 gelu (tanh form)
+// the activation of a gated unit: 0 silu, 1 relu, 2 gelu (tanh form); 3, the clamped unit: min(gate, limit) times the
+// sigmoid of slope times it, times (up kept within +-limit) + shift
+struct GluClamp {
+    float limit, slope, shift;
+};
 __device__ __forceinline__ float glu_act(float g, int act) {
     if (act == 1) return fmaxf(g, 0.f);
     if (act == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
@@ -283,7 +432,7 @@ __device__ __forceinline__ float glu_act(float g, int act) {
 }
 
 template <typename A>
-__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ a, int F, int block, size_t total, int act) {
+__global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ a, int F, int block, size_t total, int act, GluClamp cl) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -294,6 +443,11 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ a, int
         const size_t uc = block ? gc + block : F + f;
         const float g = to_f32<A>(gu[t * 2 * F + gc]);
         const float u = to_f32<A>(gu[t * 2 * F + uc]);
+        if (act == 3) {
+            const float gc_ = fminf(g, cl.limit), uc_ = fminf(fmaxf(u, -cl.limit), cl.limit);
+            a[i] = from_f32<A>(gc_ / (1.0f + expf(-cl.slope * gc_)) * (uc_ + cl.shift));
+            continue;
+        }
         a[i] = from_f32<A>(glu_act(g, act) * u);
     }
 }
@@ -301,7 +455,7 @@ __global__ void silu_mul_kernel(const A* __restrict__ gu, A* __restrict__ a, int
 // Eight outputs per thread with 16-byte accesses (bfloat16) when F and the group size are
 // multiples of 8.
 __global__ void silu_mul_vec8_kernel(const bf16* __restrict__ gu, bf16* __restrict__ a, int F, int block,
-                                     size_t total8, int act) {
+                                     size_t total8, int act, GluClamp cl) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -322,13 +476,17 @@ __global__ void silu_mul_vec8_kernel(const bf16* __restrict__ gu, bf16* __restri
         for (int j = 0; j < 8; ++j) {
             // sigmoid by ex2.approx and rcp.approx (relative error about 1e-6, far below the bf16 rounding of
             // the result): with expf and a division the kernel was bound by instruction issue, not by memory
-            const float g = __bfloat162float(ge[j]), u = __bfloat162float(ue[j]);
-            if (act) {
+            float g = __bfloat162float(ge[j]), u = __bfloat162float(ue[j]);
+            if (act == 1 || act == 2) {
                 oe[j] = __float2bfloat16_rn(glu_act(g, act) * u);
                 continue;
             }
+            if (act == 3) {
+                g = fminf(g, cl.limit);
+                u = fminf(fmaxf(u, -cl.limit), cl.limit) + cl.shift;
+            }
             float e, r;
-            asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * -1.4426950408889634f));
+            asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * (act == 3 ? cl.slope * -1.4426950408889634f : -1.4426950408889634f)));
             asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
             oe[j] = __float2bfloat16_rn((g * r) * u);
         }
@@ -336,8 +494,10 @@ __global__ void silu_mul_vec8_kernel(const bf16* __restrict__ gu, bf16* __restri
     }
 }
 
-extern "C" int aie_silu_mul(const void* gu, void* a, int dtype, int T, int F, int block, int act, cudaStream_t stream) {
-    if (block < 0 || (block && F % block) || act < 0 || act > 2) return AIE_BAD_ARG;
+extern "C" int aie_silu_mul(const void* gu, void* a, int dtype, int T, int F, int block, int act, float limit, float slope,
+                            float shift, cudaStream_t stream) {
+    if (block < 0 || (block && F % block) || act < 0 || act > 3) return AIE_BAD_ARG;
+    const GluClamp cl{limit, slope, shift};
     if (T <= 0) return 0;
     const size_t total = (size_t)T * F;
     int blocks = (int)((total + 255) / 256);
@@ -346,13 +506,13 @@ extern "C" int aie_silu_mul(const void* gu, void* a, int dtype, int T, int F, in
         const size_t total8 = total / 8;
         int b8 = (int)((total8 + 255) / 256);
         if (b8 > aie_sm_count() * 16) b8 = aie_sm_count() * 16;
-        launch_pdl(silu_mul_vec8_kernel, dim3(b8), dim3(256), 0, stream, (const bf16*)gu, (bf16*)a, F, block, total8, act);
+        launch_pdl(silu_mul_vec8_kernel, dim3(b8), dim3(256), 0, stream, (const bf16*)gu, (bf16*)a, F, block, total8, act, cl);
         AIE_LAUNCH_CHECK();
     }
     if (dtype == AIE_F32)
-        launch_pdl(silu_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)a, F, block, total, act);
+        launch_pdl(silu_mul_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)a, F, block, total, act, cl);
     else if (dtype == AIE_BF16)
-        launch_pdl(silu_mul_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, (bf16*)a, F, block, total, act);
+        launch_pdl(silu_mul_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, (bf16*)a, F, block, total, act, cl);
     else
         return AIE_BAD_ARG;
     AIE_LAUNCH_CHECK();

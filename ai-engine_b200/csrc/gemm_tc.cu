@@ -79,6 +79,12 @@ struct TcRope {
     int bt_width, num_pages, P, H, K, d, write;
 };
 
+// The gated unit of the SWIGLU epilogue: min(gate, limit) * sigmoid(slope * it) * (up kept within +-limit + shift);
+// silu(gate) * up is limit = infinity, slope 1, shift 0.
+struct TcGlu {
+    float limit, slope, shift;
+};
+
 __device__ __forceinline__ unsigned cluster_rank() {
     unsigned r;
     asm volatile("mov.u32 %0, %%cluster_ctarank;\n" : "=r"(r));
@@ -112,7 +118,7 @@ template <int BN, int EPI, typename OT>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                OT* __restrict__ C, int T, int N, int K, int ldc, int kb_per_split, int STAGES, int raw_parts,
-               unsigned* err, const TcRope rope, const int* __restrict__ tile_w) {
+               unsigned* err, const TcRope rope, const int* __restrict__ tile_w, const TcGlu glu) {
     constexpr int TMEM_COLS = BN < 32 ? 32 : BN;
     // grouped rows: token tile y multiplies the weight tile_w[y] of a stack of [N, K] weights (-1: an empty tile).
     // The list is the previous kernel's output, so it is read behind the dependency wait.
@@ -306,13 +312,17 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 if (EPI == TC_EPI_STORE) {
                     out = sum_peers(tile_addr + (tt * TC_BM + j) * 4, parts);
                 } else {     // rows 0..63 of the tile are gate rows, rows 64..127 their up rows
-                    const float g = sum_peers(tile_addr + (tt * TC_BM + j) * 4, parts);
-                    const float u = sum_peers(tile_addr + (tt * TC_BM + 64 + j) * 4, parts);
+                    float g = sum_peers(tile_addr + (tt * TC_BM + j) * 4, parts);
+                    float u = sum_peers(tile_addr + (tt * TC_BM + 64 + j) * 4, parts);
+                    if (glu.limit < INFINITY) {
+                        g = fminf(g, glu.limit);
+                        u = fminf(fmaxf(u, -glu.limit), glu.limit);
+                    }
                     // sigmoid by ex2.approx and rcp.approx (relative error about 1e-6; the result is rounded to bf16)
                     float e, r;
-                    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * -1.4426950408889634f));
+                    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(g * (glu.slope * -1.4426950408889634f)));
                     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-                    out = (g * r) * u;
+                    out = (g * r) * (u + glu.shift);
                 }
                 if (f0 + j < width) tc_store<OT>(C + (size_t)(t0 + tt) * ldc + f0 + j, out);
             }
@@ -345,7 +355,7 @@ static int make_map(CUtensorMap* map, const void* ptr, int rows, int K, int box_
 template <int BN, int EPI, typename OT>
 static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* C, int T, int N, int K, int ldc,
                      int splits, int raw_parts, unsigned* err, cudaStream_t st, const TcRope& rope = TcRope(),
-                     const int* tile_w = nullptr) {
+                     const int* tile_w = nullptr, const TcGlu glu = TcGlu{INFINITY, 1.f, 0.f}) {
     const int kb_total = (K + TC_BK - 1) / TC_BK;
     const int kbps = (kb_total + splits - 1) / splits;
     auto kern = gemm_tc_kernel<BN, EPI, OT>;
@@ -380,17 +390,20 @@ static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* C, int 
     }
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, kern, mw, mx, (OT*)C, T, N, K, ldc, kbps, stages, raw_parts, err, rope, tile_w);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, kern, mw, mx, (OT*)C, T, N, K, ldc, kbps, stages, raw_parts, err, rope, tile_w, glu);
     return (int)e;
 }
 
 // bn: token tile (16, 32, 64, 128, 256).  splits: parts of K: 1 .. 8 joined in a cluster, or, with
 // raw_parts (float32 output only, no swiglu), any number stored one after the other: C is [splits, T, N].
-// swiglu: W is [2F, K] in 128-row tiles of 64 gate rows + their 64 up rows (N = 2F), C is [T, F].
+// swiglu: W is [2F, K] in 128-row tiles of 64 gate rows + their 64 up rows (N = 2F), C is [T, F]; limit, slope and
+// shift are those of the gated unit (TcGlu).
 // Requires K % 8 == 0 (16-byte rows) and 16-byte aligned X and W.
 extern "C" int aie_gemm_tc(const void* X, const void* W, void* C, int out_dtype, int T, int N, int K, int ldc,
-                           int bn, int splits, int swiglu, int raw_parts, unsigned* err, cudaStream_t stream) {
+                           int bn, int splits, int swiglu, int raw_parts, float limit, float slope, float shift,
+                           unsigned* err, cudaStream_t stream) {
     if (T <= 0 || N <= 0) return 0;
+    const TcGlu glu{limit, slope, shift};
     if (K <= 0 || K % 8 || ((size_t)X & 15) || ((size_t)W & 15)) return AIE_UNSUPPORTED;
     if (splits < 1 || (!raw_parts && splits > 8) || splits > 65535) return AIE_BAD_ARG;
     if (raw_parts && (swiglu || out_dtype != AIE_F32)) return AIE_BAD_ARG;
@@ -404,8 +417,8 @@ extern "C" int aie_gemm_tc(const void* X, const void* W, void* C, int out_dtype,
     if (rc) return rc;
 #define GO(BNV)                                                                                                   \
     if (swiglu)                                                                                                   \
-        rc = out_dtype == AIE_BF16 ? launch_tc<BNV, TC_EPI_SWIGLU, bf16>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream)  \
-                                   : launch_tc<BNV, TC_EPI_SWIGLU, float>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream); \
+        rc = out_dtype == AIE_BF16 ? launch_tc<BNV, TC_EPI_SWIGLU, bf16>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream, TcRope(), nullptr, glu)  \
+                                   : launch_tc<BNV, TC_EPI_SWIGLU, float>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream, TcRope(), nullptr, glu); \
     else                                                                                                          \
         rc = out_dtype == AIE_BF16 ? launch_tc<BNV, TC_EPI_STORE, bf16>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream)   \
                                    : launch_tc<BNV, TC_EPI_STORE, float>(mw, mx, C, T, N, K, ldc, splits, raw_parts, err, stream)

@@ -5,6 +5,8 @@
 //   i reads j  iff  j <= i and (window <= 0 or i - j < window or j < keep_first)
 //   out_i = gate[i, h] * sum_j exp(s(i, j)) v_j / (exp(sink[h]) + sum_j exp(s(i, j)))
 //
+// cap > 0: (q_i . k_j) * scale * temp[h] is replaced by cap * tanh(it / cap).  gate_logits: every output element is
+// multiplied by the sigmoid of a logit of its own.  tied: values are the keys, and a row is that one vector of d == e.
 // The sink is a term of the denominator that has no key and no value.  Scores, weights and sums are float32.
 // chunk > 0 (without a window): i reads j  iff  j <= i and j / chunk == i / chunk.
 // maps > 1: a key/value head has `maps` keys in front of its one value, a row is [k_0 .. k_(maps-1) | v]; query head h
@@ -19,7 +21,8 @@
 //                        elements of every head (neighbouring pairs, or halves), mixes the value with another
 //                        layer's value of the same token, and writes q and the cache row [k | v].  With
 //                        `per_head` every head (and map) of q and k is normed by itself, with one weight of d
-//                        elements for all of them.
+//                        elements for all of them; with `unit` every head is divided by its root mean square behind
+//                        the rotation, without a weight.
 //   sink_attention_plain one block per (query token, head), any sizes up to 256; keys are walked in chunks of
 //                        128 that start at multiples of 128 of the absolute key position, so the order of
 //                        every addition depends on the query's position only.
@@ -198,21 +201,23 @@ normed_attn_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
     }
 }
 
-// The same for heads that are normed one by one, not rotated and not mixed: a warp per head of q, k or v, a head's
-// elements in registers (d <= 256).
+// The same for heads that are normed one by one (or not), rotated in neighbouring pairs (or not) and not mixed: a warp
+// per head of q, k or v, a head's elements in registers (d <= 256).  A norm with weights comes ahead of the rotation,
+// `unit` behind it; rotated elements are multiplied by `mag`.
 template <typename A>
 __global__ void __launch_bounds__(256)
 head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias,
-                           const float* __restrict__ q_w, const float* __restrict__ k_w, float eps, A* __restrict__ q_out,
+                           const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                           const float* __restrict__ inv_freq, int rot_dims, float mag, int unit, A* __restrict__ q_out,
                            A* __restrict__ pages, const int* __restrict__ positions, const int* __restrict__ token_req,
                            const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
-                           int e, int maps, int write, unsigned* err) {
+                           int e, int maps, int tied, int write, unsigned* err) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int K = G * maps, nq = H * d, nk = K * d;
     const int hh = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);      // heads of q, then of k, then of v
-    if (hh >= H + K + G || (hh >= H && !write)) return;
+    if (hh >= H + K + (tied ? 0 : G) || (hh >= H && !write)) return;
     const bool is_v = hh >= H + K;
     const int n = is_v ? e : d;
     const int at = is_v ? nq + nk + (hh - H - K) * e : hh * d;
@@ -227,7 +232,7 @@ head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
             return;
         }
         const int k = hh - H, g = is_v ? k - K : k / maps;
-        dst = pages + (((size_t)page * G + g) * P + (pos - pidx * P)) * (maps * d + e) + (is_v ? maps * d : (k % maps) * d);
+        dst = pages + (((size_t)page * G + g) * P + (pos - pidx * P)) * (maps * d + (tied ? 0 : e)) + (is_v ? maps * d : (k % maps) * d);
     }
     float x[8], ss = 0.f;
 #pragma unroll
@@ -236,29 +241,68 @@ head_normed_prepare_kernel(const float* __restrict__ proj, int ld, const float* 
         x[i] = c < n ? row[c] + (b ? b[c] : 0.f) : 0.f;
         ss += x[i] * x[i];
     }
-    float inv = 1.f;
     const float* w = is_v ? nullptr : (hh < H ? q_w : k_w);
-    if (w) inv = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+    if (w) {
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int c = lane + 32 * i;
+            if (c < n) x[i] = (x[i] * inv) * w[c];
+        }
+    }
+    if (rot_dims > 0 && !is_v) {                        // the other element of a pair is the neighbouring lane's
+        const float pos = (float)positions[t];
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int c = lane + 32 * i;
+            const float other = __shfl_xor_sync(0xffffffffu, x[i], 1);
+            if (c < rot_dims) {
+                float sn, cs;
+                sincosf(pos * inv_freq[c >> 1], &sn, &cs);
+                sn *= mag;
+                cs *= mag;
+                x[i] = (c & 1) ? x[i] * cs + other * sn : x[i] * cs - other * sn;
+            }
+            ss += x[i] * x[i];
+        }
+    }
+    if (unit && !is_v) {
+        const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)d + eps);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) x[i] *= inv;
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         const int c = lane + 32 * i;
-        if (c < n) dst[c] = from_f32<A>(w ? (x[i] * inv) * w[c] : x[i]);
+        if (c < n) dst[c] = from_f32<A>(x[i]);
     }
 }
 
 // The same for sizes in steps of 4 (d <= 128): groups of L lanes (a power of two, L >= d / 4) hold a head of q or k,
-// four elements a lane; the last blocks copy the values.
+// four elements (two pairs) a lane; the last blocks copy the values.  A block makes a token's angles once, in shared
+// memory (rot_dims <= 128).
 template <typename A>
 __global__ void __launch_bounds__(256)
 head_normed_prepare4_kernel(const float* __restrict__ proj, int ld, const float* __restrict__ bias,
-                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps, A* __restrict__ q_out,
+                            const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
+                            const float* __restrict__ inv_freq, int rot_dims, float mag, int unit, A* __restrict__ q_out,
                             A* __restrict__ pages, const int* __restrict__ positions, const int* __restrict__ token_req,
                             const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G, int d,
-                            int e, int maps, int L, int head_blocks, int write, unsigned* err) {
+                            int e, int maps, int L, int head_blocks, int tied, int write, unsigned* err) {
+    __shared__ float2 turn[64];                          // (cos, sin) of the token's angles, times mag
     pdl_launch_dependents();
+    if (rot_dims > 0 && blockIdx.y < head_blocks) {      // positions and frequencies are no kernel's output
+        for (int j = threadIdx.x; j < rot_dims / 2; j += blockDim.x) {
+            float sn, cs;
+            sincosf((float)positions[blockIdx.x] * inv_freq[j], &sn, &cs);
+            turn[j] = make_float2(cs * mag, sn * mag);
+        }
+        __syncthreads();
+    }
     pdl_wait();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
-    const int K = G * maps, nq = H * d, nk = K * d, w_row = maps * d + e;
+    const int K = G * maps, nq = H * d, nk = K * d, w_row = maps * d + (tied ? 0 : e);
     const float* row = proj + (size_t)t * ld;
     A* base = nullptr;                                   // the token's place in the page, of key/value head 0
     const bool values = blockIdx.y >= head_blocks;
@@ -298,6 +342,24 @@ head_normed_prepare4_kernel(const float* __restrict__ proj, int ld, const float*
         const float inv = 1.0f / sqrtf(ss / (float)d + eps);
         x = make_float4((x.x * inv) * w.x, (x.y * inv) * w.y, (x.z * inv) * w.z, (x.w * inv) * w.w);
     }
+    if (on && c < rot_dims) {
+        const float2 a = turn[c >> 1];
+        const float u = x.x, v = x.y;
+        x.x = u * a.x - v * a.y;
+        x.y = v * a.x + u * a.y;
+        if (c + 2 < rot_dims) {
+            const float2 b = turn[(c >> 1) + 1];
+            const float u2 = x.z, v2 = x.w;
+            x.z = u2 * b.x - v2 * b.y;
+            x.w = v2 * b.x + u2 * b.y;
+        }
+    }
+    if (unit) {
+        float ss = x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+        for (int o = L >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float inv = 1.0f / sqrtf(ss / (float)d + eps);
+        x = make_float4(x.x * inv, x.y * inv, x.z * inv, x.w * inv);
+    }
     if (!on) return;
     if (hh < H) {
         store4<A>(q_out + (size_t)t * nq + hh * d + c, x);
@@ -308,9 +370,9 @@ head_normed_prepare4_kernel(const float* __restrict__ proj, int ld, const float*
 }
 
 extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* bias, const float* q_w, const float* k_w,
-                                       float eps, const float* inv_freq, int rot_dims, int halves, const float* mix_from,
-                                       const float* lambda, float* v_keep, void* q_out, void* pages, int dtype,
-                                       const int* positions, const int* token_req, const int* block_table, int bt_width,
+                                       float eps, const float* inv_freq, int rot_dims, int halves, float mag, int unit,
+                                       int tied, const float* mix_from, const float* lambda, float* v_keep,
+                                       void* q_out, void* pages, int dtype, const int* positions, const int* token_req, const int* block_table, int bt_width,
                                        int num_pages, int P, int T, int H, int G, int d, int e, int maps, int per_head,
                                        int write, unsigned* err, cudaStream_t stream) {
     if (T <= 0) return 0;
@@ -318,28 +380,30 @@ extern "C" int aie_normed_attn_prepare(const float* proj, int ld, const float* b
     if (H <= 0 || G <= 0 || H % G || d <= 0 || e <= 0 || rot_dims < 0 || rot_dims > d || rot_dims % 2 ||
         (mix_from && !lambda) || (q_w && !k_w) || (rot_dims > 0 && !inv_freq))
         return AIE_BAD_ARG;
-    if ((per_head || !q_w) && rot_dims == 0 && !mix_from && !v_keep && d <= 256 && e <= 256) {
+    if (tied && (d != e || maps != 1)) return AIE_BAD_ARG;
+    if ((per_head || !q_w) && (rot_dims == 0 || !halves) && !mix_from && !v_keep && d <= 256 && e <= 256) {
         const size_t al = (size_t)proj | (size_t)bias | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)pages;
         if (d % 4 == 0 && e % 4 == 0 && ld % 4 == 0 && d <= 128 && !(al & 15) && (dtype == AIE_F32 || dtype == AIE_BF16)) {
             int L = 1;
             while (L * 4 < d) L *= 2;
-            const int hb = (H + G * maps + 8 * (32 / L) - 1) / (8 * (32 / L)), vb = (G * e / 4 + 255) / 256;
+            const int hb = (H + G * maps + 8 * (32 / L) - 1) / (8 * (32 / L)), vb = tied ? 0 : (G * e / 4 + 255) / 256;
             const dim3 grid4(T, hb + vb);
             if (dtype == AIE_F32)
-                launch_pdl(head_normed_prepare4_kernel<float>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, write, err);
+                launch_pdl(head_normed_prepare4_kernel<float>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, mag, unit, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, tied, write, err);
             else
-                launch_pdl(head_normed_prepare4_kernel<bf16>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, write, err);
+                launch_pdl(head_normed_prepare4_kernel<bf16>, grid4, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, mag, unit, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, L, hb, tied, write, err);
             AIE_LAUNCH_CHECK();
         }
         const dim3 grid(T, (H + G * maps + G + 7) / 8);
         if (dtype == AIE_F32)
-            launch_pdl(head_normed_prepare_kernel<float>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+            launch_pdl(head_normed_prepare_kernel<float>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, mag, unit, (float*)q_out, (float*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, tied, write, err);
         else if (dtype == AIE_BF16)
-            launch_pdl(head_normed_prepare_kernel<bf16>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, write, err);
+            launch_pdl(head_normed_prepare_kernel<bf16>, grid, dim3(256), 0, stream, proj, ld, bias, q_w, k_w, eps, inv_freq, rot_dims, mag, unit, (bf16*)q_out, (bf16*)pages, positions, token_req, block_table, bt_width, num_pages, P, H, G, d, e, maps, tied, write, err);
         else
             return AIE_BAD_ARG;
         AIE_LAUNCH_CHECK();
     }
+    if (mag != 1.f || unit || tied) return AIE_UNSUPPORTED;
     const size_t smem = ((size_t)(H + G * maps) * d + 32) * sizeof(float);
     if (smem > 200 * 1024) return AIE_UNSUPPORTED;
 #define AIE_NAP(A)                                                                                                    \
@@ -367,7 +431,8 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
                             const float* __restrict__ slope, const float* __restrict__ sink,
                             const int* __restrict__ positions, const int* __restrict__ token_req,
                             const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G,
-                            int d, int e, int window, int keep_first, int chunk, int maps, float scale,
+                            int d, int e, int window, int keep_first, int chunk, int maps, float scale, float cap,
+                            int tied, const float* __restrict__ gate_logits, int ld_gate,
                             const int* __restrict__ token_list, unsigned* err) {
     extern __shared__ __align__(16) float sm[];
     float* q_s = sm;                                  // d (rounded up to even)
@@ -379,7 +444,7 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
     const int pos = positions[t];
     const int row = token_req[t];
     const int g = h / (H / G);
-    const int w = maps * d + e, k_off = (h % maps) * d, v_off = maps * d;
+    const int w = maps * d + (tied ? 0 : e), k_off = (h % maps) * d, v_off = tied ? 0 : maps * d;
     const float qs = scale * (temp ? temp[h] : 1.f), sl = slope ? slope[h] : 0.f;
     for (int c = tid; c < d; c += blockDim.x) q_s[c] = to_f32<A>(q[((size_t)t * H + h) * d + c]);
     __syncthreads();
@@ -412,7 +477,9 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
                 const C* kr = pages + off + k_off;
                 float dot = 0.f;
                 for (int c = 0; c < d; ++c) dot += q_s[c] * to_f32<C>(kr[c]);
-                s = dot * qs - sl * (float)(pos - kp);
+                s = dot * qs;
+                if (cap > 0.f) s = cap * tanhf(s / cap);
+                s -= sl * (float)(pos - kp);
             }
         }
         off_s[tid] = off;
@@ -438,16 +505,20 @@ sink_attention_plain_kernel(const A* __restrict__ q, const C* __restrict__ pages
     }
     const float inv = (l > 0.f ? 1.0f / l : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
     O* o = out + ((size_t)t * H + h) * e;
-    if (tid < e) o[tid] = from_f32<O>(acc0 * inv);
-    if (tid + SA_CHUNK < e) o[tid + SA_CHUNK] = from_f32<O>(acc1 * inv);
+    const float* gl = gate_logits ? gate_logits + (size_t)t * ld_gate + (size_t)h * e : nullptr;
+    if (tid < e) o[tid] = from_f32<O>(acc0 * inv * (gl ? 1.f / (1.f + expf(-gl[tid])) : 1.f));
+    if (tid + SA_CHUNK < e)
+        o[tid + SA_CHUNK] = from_f32<O>(acc1 * inv * (gl ? 1.f / (1.f + expf(-gl[tid + SA_CHUNK])) : 1.f));
 }
 
 extern "C" int aie_sink_attention_plain(const void* q, const void* pages, void* out, int dtype, int out_dtype, const float* gate,
                                         const float* temp, const float* slope, const float* sink, const int* positions,
                                         const int* token_req, const int* block_table, int bt_width, int num_pages,
                                         int P, int T, int H, int G, int d, int e, int window, int keep_first,
-                                        int chunk, int maps, float scale, const int* token_list, unsigned* err, cudaStream_t stream) {
+                                        int chunk, int maps, float scale, float cap, int tied, const float* gate_logits,
+                                        int ld_gate, const int* token_list, unsigned* err, cudaStream_t stream) {
     if (T <= 0) return 0;
+    if (tied && (d != e || maps != 1)) return AIE_BAD_ARG;
     if (d <= 0 || d > 2 * SA_CHUNK || e <= 0 || e > 2 * SA_CHUNK || G <= 0 || H % G || H > 65535) return AIE_UNSUPPORTED;
     if (maps < 1 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     const size_t smem = (size_t)(((d + 1) & ~1) + SA_CHUNK + 32) * sizeof(float) + SA_CHUNK * sizeof(long long);
@@ -455,7 +526,7 @@ extern "C" int aie_sink_attention_plain(const void* q, const void* pages, void* 
 #define AIE_SA(A, O)                                                                                                   \
     sink_attention_plain_kernel<A, A, O><<<grid, SA_CHUNK, smem, stream>>>(                                            \
         (const A*)q, (const A*)pages, (O*)out, gate, temp, slope, sink, positions, token_req, block_table, bt_width,   \
-        num_pages, P, H, G, d, e, window, keep_first, chunk, maps, scale, token_list, err)
+        num_pages, P, H, G, d, e, window, keep_first, chunk, maps, scale, cap, tied, gate_logits, ld_gate, token_list, err)
     if (dtype == AIE_F32 && out_dtype == AIE_F32) AIE_SA(float, float);
     else if (dtype == AIE_BF16 && out_dtype == AIE_BF16) AIE_SA(bf16, bf16);
     else if (dtype == AIE_BF16 && out_dtype == AIE_F32) AIE_SA(bf16, float);

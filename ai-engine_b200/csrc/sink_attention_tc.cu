@@ -1,11 +1,16 @@
 // bfloat16 attention with a distance bias, a window that keeps the first tokens, a sink and a gate per head on
 // tensor cores (mma.sync m16n8k16, bf16 in, float32 accumulate), over a paged cache of one plane whose rows hold
-// a key (DK elements) and behind it a value (DV elements); DK and DV each 32, 64 or 128.
+// a key (d elements) and behind it a value (e elements).  The kernels are compiled for keys of DK and values of DV
+// elements, each 32, 64 or 128; d <= DK and e <= DV in steps of 8 (what is missing is filled with zeros in shared
+// memory).
 //
 //   s(i, j) = (q_i . k_j) * scale * temp[h] - slope[h] * (i - j)
 //   i reads j  iff  j <= i and (window <= 0 or i - j < window or j < keep_first)
 //   out_i = gate[i, h] * sum_j exp(s(i, j)) v_j / (exp(sink[h]) + sum_j exp(s(i, j)))
 //
+// cap > 0: (q_i . k_j) * scale * temp[h] is replaced by cap * tanh(it / cap).  gate_logits: every output element is
+// multiplied by the sigmoid of a logit of its own.  TIED: values are the keys, a row is that one vector (d == e), and a
+// tile of rows is loaded once for both products.
 // chunk > 0 (without a window): i reads j  iff  j <= i and j / chunk == i / chunk.
 // maps > 1: a key/value head has `maps` keys in front of its one value, a row is [k_0 .. k_(maps-1) | v]; query head h
 // of the H (all maps counted) reads key h % maps of key/value head h / (H / G).  The prompt kernel's CTA loads the one
@@ -40,6 +45,12 @@ template <int D> __device__ __forceinline__ bf16* sk_at(bf16* base, int row, int
     return base + row * D + ((chunk ^ ((row >> 1) & 3)) << 3);
 }
 
+// cap * tanh(v / cap) as cap (1 - 2 / (1 + e^(2 v / cap))): an absolute error of some 1e-7 cap, right at both ends
+__device__ __forceinline__ float sk_bounded(float v, float cap, float two_over_cap) {
+    return cap - __fdividef(2.f * cap, 1.f + __expf(v * two_over_cap));
+}
+__device__ __forceinline__ float sk_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
 // One warp, 16 query rows against a tile of N keys in shared memory.  The thread holds rows (lane / 4) and
 // (lane / 4) + 8: their positions qp, the first keys low that they read, factors qs (scale * temp) and slopes sl.  `masked`: apply the visibility
 // rule (tiles wholly inside every row's sight skip it); keys above `key_end` are never visible.
@@ -47,7 +58,7 @@ template <int DK, int DV, int N>
 __device__ __forceinline__ void sk_tile(const bf16* kb, const bf16* vb, const unsigned (&qf)[DK / 16][4],
                                         float (&o)[DV / 8][4], float (&m_run)[2], float (&l_run)[2], int kbase,
                                         const int (&qp)[2], const int (&low)[2], const float (&qs)[2],
-                                        const float (&sl)[2], int keep_first, bool masked, int lane) {
+                                        const float (&sl)[2], int keep_first, bool masked, float cap, int lane) {
     float s[N / 8][4];
 #pragma unroll
     for (int j = 0; j < N / 8; ++j)
@@ -65,13 +76,22 @@ __device__ __forceinline__ void sk_tile(const bf16* kb, const bf16* vb, const un
         }
     }
     float tmax[2] = {-INFINITY, -INFINITY};
+    float qf_[2] = {qs[0], qs[1]};
+    if (cap > 0.f) {
+        const float tc = 2.f / cap;
+#pragma unroll
+        for (int j = 0; j < N / 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s[j][e] = sk_bounded(s[j][e] * qs[e >> 1], cap, tc);
+        qf_[0] = qf_[1] = 1.f;
+    }
 #pragma unroll
     for (int j = 0; j < N / 8; ++j) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int i = e >> 1;
             const int key = kbase + j * 8 + 2 * (lane & 3) + (e & 1);
-            float v = s[j][e] * qs[i] - sl[i] * (float)(qp[i] - key);
+            float v = s[j][e] * qf_[i] - sl[i] * (float)(qp[i] - key);
             if (masked) {
                 const bool ok = key <= qp[i] && (key >= low[i] || key < keep_first);
                 if (!ok) v = -INFINITY;
@@ -141,21 +161,21 @@ __device__ __forceinline__ int sk_low(int pos, int window, int chunk) {
     return window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0;
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool TIED>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, bf16* __restrict__ out,
                     const float* __restrict__ gate, const float* __restrict__ temp, const float* __restrict__ slope,
                     const float* __restrict__ sink, const int* __restrict__ tiles, const int* __restrict__ q_start,
                     const int* __restrict__ q_len, const int* __restrict__ ctx_len,
                     const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int G,
-                    int window, int keep_first, int chunk, int maps, float scale, float* __restrict__ out32,
-                    unsigned* err) {
+                    int d, int e, int window, int keep_first, int chunk, int maps, float scale, float cap,
+                    const float* __restrict__ gate_logits, int ld_gate, float* __restrict__ out32, unsigned* err) {
     constexpr int N = 64;
-    constexpr int CK = DK / 8, CW = (DK + DV) / 8;           // 16-byte pieces of a key; of a key and a value
+    constexpr int CK = DK / 8, CW = TIED ? CK : (DK + DV) / 8;      // 16-byte pieces of a key; of a key and a value
     extern __shared__ __align__(128) unsigned char smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);            // [128][DK]
     bf16* k_s = q_s + SK_M * DK;                               // [2][64][DK]
-    bf16* v_s = k_s + 2 * N * DK;                              // [2][64][DV]
+    bf16* v_s = TIED ? k_s : k_s + 2 * N * DK;                 // [2][64][DV]
     int* row_s = reinterpret_cast<int*>(v_s + 2 * N * DV);     // [2][64] cache rows of the tile's keys
 
     pdl_launch_dependents();
@@ -164,8 +184,9 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
     const int tile_i = (int)gridDim.y - 1 - (int)blockIdx.y;   // the list holds the tiles fewest keys first
     const int r = tiles[2 * tile_i], q_off = tiles[2 * tile_i + 1];
     const int h = blockIdx.x, g = h / (H / G);
-    const int W = maps * DK + DV;                              // elements of a cache row
-    const int k_off = (h % maps) * DK, v_off = (maps - 1) * DK;      // of this head's key; of the value behind c * 8 >= DK
+    const int W = maps * d + (TIED ? 0 : e);                   // elements of a cache row
+    const int k_off = (h % maps) * d, v_off = maps * d - DK;   // of this head's key; of the value behind c * 8 >= DK
+    const int ck = d / 8, cv = CK + e / 8;                     // pieces that a row has: c < ck of the key, CK <= c < cv
     const int t0 = q_start[r] + q_off;
     const int rows_valid = min(SK_M, q_len[r] - q_off);
     const int p0 = ctx_len[r] + q_off;              // position of the tile's first query
@@ -174,8 +195,8 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
 
     for (int i = tid; i < SK_M * CK; i += SK_WARPS * 32) {
         const int row = i / CK, c = i % CK;
-        const bool ok = row < rows_valid;
-        cp_async16(sk_at<DK>(q_s, row, c), q + ((size_t)(t0 + (ok ? row : 0)) * H + h) * DK + c * 8, ok);
+        const bool ok = row < rows_valid && c < ck;
+        cp_async16(sk_at<DK>(q_s, row, c), q + ((size_t)(t0 + (ok ? row : 0)) * H + h) * d + (ok ? c : 0) * 8, ok);
     }
     cp_async_commit();
 
@@ -204,8 +225,8 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
         for (int i = tid; i < N * CW; i += SK_WARPS * 32) {
             const int row = i / CW, c = i % CW;
             const int prow = row_s[buf * N + row];
-            const bool ok = prow >= 0;
-            const bf16* src = pages + (size_t)(ok ? prow : 0) * W + c * 8 + (c < CK ? k_off : v_off);
+            const bool ok = prow >= 0 && (c < CK ? c < ck : c < cv);
+            const bf16* src = ok ? pages + (size_t)prow * W + c * 8 + (c < CK ? k_off : v_off) : pages;
             if (c < CK) cp_async16(sk_at<DK>(kd, row, c), src, ok);
             else cp_async16(sk_at<DV>(vd, row, c - CK), src, ok);
         }
@@ -218,7 +239,7 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
+        for (int k = 0; k < 4; ++k) o[j][k] = 0.f;
     // the sink opens the running softmax: a weight exp(sink - m) = 1 at m = sink, with no value
     float m_run[2], l_run[2];
     m_run[0] = m_run[1] = sink ? sink[h] : -INFINITY;
@@ -255,7 +276,7 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
         // the rule is applied on tiles that touch the diagonal or the low edge of some row's window
         const bool masked = (kbase + N - 1 > p0) || kbase < lo_last;
         sk_tile<DK, DV, N>(k_s + buf * N * DK, v_s + buf * N * DV, qf, o, m_run, l_run, kbase, qp, low, qs, sl,
-                           keep_first, masked, lane);
+                           keep_first, masked, cap, lane);
         __syncthreads();     // everyone is done with this buffer before it is loaded again
     }
 
@@ -264,17 +285,26 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
         const int row = warp * 16 + (lane >> 2) + i * 8;
         if (row >= rows_valid) continue;
         const float inv = (l_run[i] > 0.f ? 1.0f / l_run[i] : 0.f) * (gate ? gate[(size_t)(t0 + row) * H + h] : 1.f);
-        if (out32) {
-            float* dst = out32 + ((size_t)(t0 + row) * H + h) * DV + 2 * (lane & 3);
+        if (gate_logits) {
+            const float* gl = gate_logits + (size_t)(t0 + row) * ld_gate + (size_t)h * e + 2 * (lane & 3);
 #pragma unroll
             for (int j = 0; j < DV / 8; ++j)
-                *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[j][i * 2] * inv, o[j][i * 2 + 1] * inv);
+                if (j * 8 < e) {
+                    o[j][i * 2] *= sk_sigmoid(gl[j * 8]);
+                    o[j][i * 2 + 1] *= sk_sigmoid(gl[j * 8 + 1]);
+                }
+        }
+        if (out32) {
+            float* dst = out32 + ((size_t)(t0 + row) * H + h) * e + 2 * (lane & 3);
+#pragma unroll
+            for (int j = 0; j < DV / 8; ++j)
+                if (j * 8 < e) *reinterpret_cast<float2*>(dst + j * 8) = make_float2(o[j][i * 2] * inv, o[j][i * 2 + 1] * inv);
             continue;
         }
-        bf16* dst = out + ((size_t)(t0 + row) * H + h) * DV + 2 * (lane & 3);
+        bf16* dst = out + ((size_t)(t0 + row) * H + h) * e + 2 * (lane & 3);
 #pragma unroll
         for (int j = 0; j < DV / 8; ++j)
-            *reinterpret_cast<unsigned*>(dst + j * 8) = pack_bf16(o[j][i * 2] * inv, o[j][i * 2 + 1] * inv);
+            if (j * 8 < e) *reinterpret_cast<unsigned*>(dst + j * 8) = pack_bf16(o[j][i * 2] * inv, o[j][i * 2 + 1] * inv);
     }
 }
 
@@ -288,27 +318,32 @@ sink_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, 
 // keys of one stage of a warp: about 8 KB of cache rows, a multiple of 16 keys
 template <int W> struct SdStage { static constexpr int keys = W > 128 ? 16 : (W > 64 ? 32 : 64); };
 
-template <int DK, int DV> struct SdSmem {
-    static constexpr int W = DK + DV, STILE = SdStage<W>::keys;
+template <int DK, int DV, bool TIED> struct SdSmem {
+    static constexpr int W = TIED ? DK : DK + DV, STILE = SdStage<W>::keys;
     static constexpr size_t stage_bytes = (size_t)STILE * W * sizeof(bf16);
     static constexpr size_t rows_off = (size_t)SD_WARPS * SD_NST * stage_bytes;
-    static constexpr size_t bytes = rows_off + (size_t)SD_WARPS * STILE * sizeof(int);
+    static constexpr size_t ring = rows_off + (size_t)SD_WARPS * STILE * sizeof(int);
+    static constexpr size_t joined = (size_t)SD_WARPS * SD_HEADS * DV * sizeof(float);      // the warps' outputs
+    static constexpr size_t bytes = ring > joined ? ring : joined;
 };
 
 // The keys a lone token at `pos` reads are numbered u = 0 .. nk-1: first the `kept` first keys that the window
 // has passed, then the window's own from `lo` on.  Every numbered key is visible, so no rule is applied to
 // them; a key's true position enters the distance bias.
-template <int DK, int DV>
+template <int DK, int DV, bool TIED>
 __global__ void __launch_bounds__(SD_WARPS * 32)
 sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, bf16* __restrict__ out,
                    float* __restrict__ part_o, float* __restrict__ part_lse, const float* __restrict__ gate,
                    const float* __restrict__ temp, const float* __restrict__ slope, const float* __restrict__ sink,
                    const int* __restrict__ dec_tokens, const int* __restrict__ positions,
                    const int* __restrict__ token_req, const int* __restrict__ block_table, int bt_width,
-                   int num_pages, int P, int H, int G, int GC, int window, int keep_first, int chunk, int maps,
-                   float scale, int S, float* __restrict__ out32, unsigned* err) {
-    constexpr int W = DK + DV, CW = W / 8, CK = DK / 8;
+                   int num_pages, int P, int H, int G, int GC, int d, int e, int window, int keep_first, int chunk,
+                   int maps, float scale, float cap, const float* __restrict__ gate_logits, int ld_gate, int S,
+                   float* __restrict__ out32, unsigned* err) {
+    constexpr int W = SdSmem<DK, DV, TIED>::W, CW = W / 8, CK = DK / 8;      // of a row in shared memory
     constexpr int STILE = SdStage<W>::keys, KS = DK / 16;
+    const int w_row = d + (TIED ? 0 : e);              // of a row in the pages; d: all keys of it
+    const int ck = d / 8, cv = CK + e / 8, v_off = d - DK;
     extern __shared__ __align__(128) unsigned char sd_smem[];
     __shared__ float mrg_m[SD_WARPS][SD_HEADS], mrg_l[SD_WARPS][SD_HEADS];
 
@@ -325,8 +360,8 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
     const int qrow = lane >> 2, qcol = (lane & 3) * 2;
     const int* bt = block_table + (size_t)row * bt_width;
 
-    bf16* stage0 = reinterpret_cast<bf16*>(sd_smem + (size_t)warp * SD_NST * SdSmem<DK, DV>::stage_bytes);
-    int* rows_w = reinterpret_cast<int*>(sd_smem + SdSmem<DK, DV>::rows_off) + warp * STILE;
+    bf16* stage0 = reinterpret_cast<bf16*>(sd_smem + (size_t)warp * SD_NST * SdSmem<DK, DV, TIED>::stage_bytes);
+    int* rows_w = reinterpret_cast<int*>(sd_smem + SdSmem<DK, DV, TIED>::rows_off) + warp * STILE;
 
     const int lo = sk_low(pos, window, chunk);
     const int kept = min(keep_first, lo);
@@ -354,15 +389,16 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
             }
             __syncwarp();
             bf16* kd = stage0 + (size_t)(i % SD_NST) * STILE * W;
-            bf16* vd = kd + STILE * DK;
+            bf16* vd = TIED ? kd : kd + STILE * DK;
 #pragma unroll
             for (int r = 0; r < STILE * CW / 32; ++r) {
                 const int idx = lane + r * 32;
                 const int kr = idx / CW, c = idx % CW;
                 const int prow = rows_w[kr];
-                const bf16* src = pages + (size_t)(prow >= 0 ? prow : 0) * W + c * 8;
-                if (c < CK) cp_async16(sk_at<DK>(kd, kr, c), src, prow >= 0);
-                else cp_async16(sk_at<DV>(vd, kr, c - CK), src, prow >= 0);
+                const bool ok = prow >= 0 && (c < CK ? c < ck : c < cv);
+                const bf16* src = ok ? pages + (size_t)prow * w_row + c * 8 + (c < CK ? 0 : v_off) : pages;
+                if (c < CK) cp_async16(sk_at<DK>(kd, kr, c), src, ok);
+                else cp_async16(sk_at<DV>(vd, kr, c - CK), src, ok);
             }
             __syncwarp();      // the rows are read before the next stage's are written
         }
@@ -376,17 +412,18 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
     unsigned qa[KS][2];
     {
         const int hh = hbase + (qrow < ng ? qrow : 0);
-        const int dm = DK / maps, k_off = (hh % maps) * dm;     // elements of a map's query; where its key lies in the row
+        const int dm = d / maps, k_off = (hh % maps) * dm;     // elements of a map's query; where its key lies in the row
         const bf16* qp = q + (size_t)t * H * dm + (size_t)hh * dm - k_off;
 #pragma unroll
         for (int ks = 0; ks < KS; ++ks) {
-            const bool on = qrow < ng && ks * 16 >= k_off && ks * 16 < k_off + dm;
-            qa[ks][0] = on ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + qcol) : 0u;
-            qa[ks][1] = on ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + 8 + qcol) : 0u;
+            const int c0 = ks * 16 - k_off;               // of this map's query; d is a multiple of 8 a map
+            qa[ks][0] = qrow < ng && c0 >= 0 && c0 < dm ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + qcol) : 0u;
+            qa[ks][1] = qrow < ng && c0 >= -8 && c0 + 8 < dm ? *reinterpret_cast<const unsigned*>(qp + ks * 16 + 8 + qcol) : 0u;
         }
     }
     const int hq = hbase + (qrow < ng ? qrow : 0);
     const float qs = scale * (temp ? temp[hq] : 1.f), sl = slope ? slope[hq] : 0.f;
+    const float tc = cap > 0.f ? 2.f / cap : 0.f;
     float m_run = -INFINITY, l_run = 0.f;
     float o[DV / 8][2];
 #pragma unroll
@@ -397,7 +434,7 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
         cp_async_wait<SD_NST - 1>();
         __syncwarp();
         bf16* kd = stage0 + (size_t)(i % SD_NST) * STILE * W;
-        bf16* vd = kd + STILE * DK;
+        bf16* vd = TIED ? kd : kd + STILE * DK;
         const int u0 = (first + i * SD_WARPS) * STILE;
         const int mid = lane >> 3;
 #pragma unroll
@@ -423,7 +460,9 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
                 for (int e = 0; e < 2; ++e) {
                     const int u = u0 + sub * 16 + j * 8 + qcol + e;
                     const int key = u < kept ? u : lo + (u - kept);
-                    sc[j][e] = u < nk ? sc[j][e] * qs - sl * (float)(pos - key) : -INFINITY;
+                    float v = sc[j][e] * qs;
+                    if (cap > 0.f) v = sk_bounded(v, cap, tc);
+                    sc[j][e] = u < nk ? v - sl * (float)(pos - key) : -INFINITY;
                     tmax = fmaxf(tmax, sc[j][e]);
                 }
             tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, 1));
@@ -478,8 +517,8 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
         }
     }
     __syncthreads();
-    for (int idx = tid; idx < ng * DV; idx += SD_WARPS * 32) {
-        const int g = idx / DV, e = idx % DV;
+    for (int idx = tid; idx < ng * e; idx += SD_WARPS * 32) {
+        const int g = idx / e, c = idx % e;
         const int h = hbase + g;
         float M = -INFINITY;
 #pragma unroll
@@ -491,18 +530,19 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
         for (int w = 0; w < SD_WARPS; ++w) {
             const float f = (mrg_m[w][g] == -INFINITY) ? 0.f : __expf(mrg_m[w][g] - M);
             L += mrg_l[w][g] * f;
-            A += mrg_o[((size_t)w * SD_HEADS + g) * DV + e] * f;
+            A += mrg_o[((size_t)w * SD_HEADS + g) * DV + c] * f;
         }
         if (whole) {
             if (sink) L += __expf(sink[h] - M);      // the sink counts once, with no value
-            const float inv = (L > 0.f ? 1.0f / L : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
-            const size_t at = ((size_t)t * H + h) * DV + e;
+            float inv = (L > 0.f ? 1.0f / L : 0.f) * (gate ? gate[(size_t)t * H + h] : 1.f);
+            if (gate_logits) inv *= sk_sigmoid(gate_logits[(size_t)t * ld_gate + (size_t)h * e + c]);
+            const size_t at = ((size_t)t * H + h) * e + c;
             if (out32) out32[at] = A * inv;
             else out[at] = __float2bfloat16_rn(A * inv);
         } else {
             const size_t pi = ((size_t)di * H + h) * S + s;
-            part_o[pi * DV + e] = L > 0.f ? A / L : 0.f;
-            if (e == 0) part_lse[pi] = L > 0.f ? M + __logf(L) : -INFINITY;
+            part_o[pi * e + c] = L > 0.f ? A / L : 0.f;
+            if (c == 0) part_lse[pi] = L > 0.f ? M + __logf(L) : -INFINITY;
         }
     }
 }
@@ -512,7 +552,8 @@ sink_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, b
 __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse,
                                  bf16* __restrict__ out, const float* __restrict__ gate,
                                  const float* __restrict__ sink, const int* __restrict__ dec_tokens, int H, int DV,
-                                 int S, float* __restrict__ out32) {
+                                 int S, const float* __restrict__ gate_logits, int ld_gate,
+                                 float* __restrict__ out32) {
     __shared__ float w_s[SD_MAX_SPLITS];
     __shared__ float wsum_s;
     pdl_launch_dependents();
@@ -541,16 +582,23 @@ __global__ void sink_join_kernel(const float* __restrict__ part_o, const float* 
         float A = 0.f;
 #pragma unroll 8
         for (int s = 0; s < S; ++s) A += w_s[s] * src[(size_t)s * DV];
+        if (gate_logits) A *= sk_sigmoid(gate_logits[(size_t)t * ld_gate + (size_t)h * DV + e]);
         const size_t at = ((size_t)t * H + h) * DV + e;
         if (out32) out32[at] = A * inv;
         else out[at] = __float2bfloat16_rn(A * inv);
     }
 }
 
+// the compiled size that holds n elements (0: none)
+static inline int sk_padded(int n) { return n <= 0 || n % 8 ? 0 : n <= 32 ? 32 : n <= 64 ? 64 : n <= 128 ? 128 : 0; }
+
 #define SK_DISPATCH(DK_, DV_, CALL)                                                        \
-    if (d == DK_ && e == DV_) { CALL(DK_, DV_) }
+    if (dk == DK_ && dv == DV_) { CALL(DK_, DV_, false) }
+#define SK_DISPATCH_TIED(D_, CALL)                                                         \
+    if (tied && dk == D_) { CALL(D_, D_, true) }
 
 #define SK_DISPATCH_ALL(CALL)                                                              \
+    SK_DISPATCH_TIED(32, CALL) else SK_DISPATCH_TIED(64, CALL) else SK_DISPATCH_TIED(128, CALL) else \
     SK_DISPATCH(32, 32, CALL) else SK_DISPATCH(32, 64, CALL) else SK_DISPATCH(32, 128, CALL) \
     else SK_DISPATCH(64, 32, CALL) else SK_DISPATCH(64, 64, CALL) else SK_DISPATCH(64, 128, CALL) \
     else SK_DISPATCH(128, 32, CALL) else SK_DISPATCH(128, 64, CALL) else SK_DISPATCH(128, 128, CALL) \
@@ -564,20 +612,23 @@ extern "C" int aie_sink_attention_prefill(const void* q, const void* pages, void
                                           int n_tiles, const int* q_start, const int* q_len, const int* ctx_len,
                                           const int* block_table, int bt_width, int num_pages, int P, int H, int G,
                                           int d, int e, int window, int keep_first, int chunk, int maps, float scale,
-                                          float* out32, unsigned* err, cudaStream_t stream) {
+                                          float cap, int tied, const float* gate_logits, int ld_gate, float* out32,
+                                          unsigned* err, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
+    const int dk = sk_padded(d), dv = sk_padded(e);
+    if ((maps > 1 && dk != d) || (tied && (d != e || maps != 1))) return AIE_BAD_ARG;
     if (maps < 1 || G <= 0 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     if (G <= 0 || H % G || n_tiles > 65535) return AIE_UNSUPPORTED;
     dim3 grid(H, n_tiles);
-#define SK_PRE(DK_, DV_)                                                                                              \
+#define SK_PRE(DK_, DV_, TIED_)                                                                                              \
     {                                                                                                                 \
-        const size_t smem = (size_t)(SK_M * DK_ + 2 * 64 * DK_ + 2 * 64 * DV_) * sizeof(bf16) + 2 * 64 * sizeof(int);   \
-        auto kern = sink_prefill_kernel<DK_, DV_>;                                                                    \
+        const size_t smem = (size_t)(SK_M * DK_ + 2 * 64 * DK_ + (TIED_ ? 0 : 2 * 64 * DV_)) * sizeof(bf16) + 2 * 64 * sizeof(int); \
+        auto kern = sink_prefill_kernel<DK_, DV_, TIED_>;                                                                    \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
         launch_pdl(kern, grid, dim3(SK_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)pages, (bf16*)out, gate, temp, slope, \
                                                     sink, tiles, q_start, q_len, ctx_len, block_table, bt_width,      \
-                                                    num_pages, P, H, G, window, keep_first, chunk, maps, scale,       \
-                                                    out32, err);                                                      \
+                                                    num_pages, P, H, G, d, e, window, keep_first, chunk, maps, scale, \
+                                                    cap, gate_logits, ld_gate, out32, err);                                                      \
     }
     SK_DISPATCH_ALL(SK_PRE)
 #undef SK_PRE
@@ -591,8 +642,11 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
                                          const int* dec_tokens, int n, const int* positions, const int* token_req,
                                          const int* block_table, int bt_width, int num_pages, int P, int H, int G,
                                          int d, int e, int window, int keep_first, int chunk, int maps, float scale,
-                                         int S, float* out32, unsigned* err, cudaStream_t stream) {
+                                         int S, float cap, int tied, const float* gate_logits, int ld_gate, float* out32,
+                                         unsigned* err, cudaStream_t stream) {
     if (n <= 0) return 0;
+    const int dk = maps > 1 ? d * maps : sk_padded(d), dv = sk_padded(e);
+    if ((maps > 1 && sk_padded(d) != d) || (tied && (d != e || maps != 1))) return AIE_BAD_ARG;
     if (maps < 1 || G <= 0 || (H / G) % maps || chunk < 0 || (chunk > 0 && (window > 0 || keep_first > 0))) return AIE_BAD_ARG;
     if (G <= 0 || H % G || S < 1 || S > SD_MAX_SPLITS || n > 65535 || (S > 1 && (!part_o || !part_lse)))
         return AIE_UNSUPPORTED;
@@ -600,15 +654,15 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
     const int gchunks = (group + GC - 1) / GC;
     if ((long long)G * gchunks > 65535) return AIE_UNSUPPORTED;
     dim3 grid(S, G * gchunks, n);
-#define SK_DEC(DK_, DV_)                                                                                              \
+#define SK_DEC(DK_, DV_, TIED_)                                                                                              \
     {                                                                                                                 \
-        const size_t smem = SdSmem<DK_, DV_>::bytes;                                                                  \
-        auto kern = sink_decode_kernel<DK_, DV_>;                                                                     \
+        const size_t smem = SdSmem<DK_, DV_, TIED_>::bytes;                                                                  \
+        auto kern = sink_decode_kernel<DK_, DV_, TIED_>;                                                                     \
         cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                           \
         launch_pdl(kern, grid, dim3(SD_WARPS * 32), smem, stream, (const bf16*)q, (const bf16*)pages, (bf16*)out, part_o, part_lse, \
                                                     gate, temp, slope, sink, dec_tokens, positions, token_req,        \
-                                                    block_table, bt_width, num_pages, P, H, G, GC, window,            \
-                                                    keep_first, chunk, maps, scale, S, out32, err);                   \
+                                                    block_table, bt_width, num_pages, P, H, G, GC, d, e, window,      \
+                                                    keep_first, chunk, maps, scale, cap, gate_logits, ld_gate, S, out32, err);                   \
     }
     d *= maps;                       // the kernel's keys are all keys of a row
     SK_DISPATCH(256, 32, SK_DEC) else SK_DISPATCH(256, 64, SK_DEC) else SK_DISPATCH(256, 128, SK_DEC) else
@@ -617,7 +671,7 @@ extern "C" int aie_sink_attention_decode(const void* q, const void* pages, void*
     if (S > 1) {
         const cudaError_t e1 = cudaGetLastError();
         if (e1 != cudaSuccess) return (int)e1;
-        launch_pdl(sink_join_kernel, dim3(n, H), dim3(128), 0, stream, part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S, out32);
+        launch_pdl(sink_join_kernel, dim3(n, H), dim3(128), 0, stream, part_o, part_lse, (bf16*)out, gate, sink, dec_tokens, H, e, S, gate_logits, ld_gate, out32);
     }
     AIE_LAUNCH_CHECK();
 }

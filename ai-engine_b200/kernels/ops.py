@@ -124,11 +124,42 @@ def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Te
     return out
 
 
-GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
+def add_rmsnorm_pair(x: torch.Tensor, delta: Optional[torch.Tensor], w1: torch.Tensor, w2: Optional[torch.Tensor],
+                     eps: float, out_dtype: torch.dtype, extra: Optional[torch.Tensor] = None,
+                     step: Optional[torch.Tensor] = None):
+    """s = x (+ delta, or the sum of its parts [parts, T, D]) (+ extra [T, D]) (+ step [D], for every row), stored into
+    the float32 stream x; (norm(s) * w1, norm(s) * w2) with norm(s) = s / sqrt(mean(s^2) + eps); w2 None: (.., None)."""
+    _dev(x, delta, w1, w2, extra, step)
+    T, D = x.shape
+    if any(t is not None and t.dtype != torch.float32 for t in (x, delta, extra, step)):
+        raise KernelError("add_rmsnorm_pair: the stream and what is added to it are float32")
+    if w1.shape != (D,) or (w2 is not None and (w2.shape != (D,) or w2.dtype != w1.dtype)) or (
+            extra is not None and extra.shape != x.shape) or (step is not None and step.shape != (D,)):
+        raise KernelError("add_rmsnorm_pair: shapes do not fit")
+    parts, stride = 0, 0
+    if delta is not None:
+        parts, stride = (delta.shape[0], delta.stride(0)) if delta.dim() == 3 else (1, 0)
+        if delta.shape[-2:] != x.shape:
+            raise KernelError("add_rmsnorm_pair: delta differs in shape from x")
+    out1 = torch.empty((T, D), dtype=out_dtype, device=x.device)
+    out2 = torch.empty((T, D), dtype=out_dtype, device=x.device) if w2 is not None else None
+    stored = any(t is not None for t in (delta, extra, step))
+    lib = library("elementwise.cu")
+    with region("add_rmsnorm_pair", (2 if stored else 1) * _nb(x) + _nb(delta, extra, out1, out2)):
+        check(lib.aie_add_rmsnorm_pair(_p(x), _p(delta), c_int(parts), c_longlong(stride), _p(extra), _p(step), _p(w1), _p(w2),
+                                       c_int(dtype_code(w1)), _p(out1), _p(out2), c_int(dtype_code(out1)), c_int(T), c_int(D),
+                                       c_float(eps), _stream()), "add_rmsnorm_pair")
+    return out1, out2
 
 
-def silu_mul(gu: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 0, activation: str = "silu") -> torch.Tensor:
-    """a[t, f] = act(gate) * up, act = silu unless `activation` names another (relu, gelu_tanh).  block == 0:
+GLU_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "clamped": 3}
+_NO_CLAMP = (float("inf"), 1.0, 0.0)      # limit, slope, shift with which the clamped unit is silu(gate) * up
+
+
+def silu_mul(gu: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 0, activation: str = "silu",
+             clamp=None) -> torch.Tensor:
+    """a[t, f] = act(gate) * up, act = silu unless `activation` names another (relu, gelu_tanh, or clamped with
+    clamp = (limit, slope, shift): g * sigmoid(slope * g) * (u + shift), g = min(gate, limit), u = up within +-limit).  block == 0:
     gu[t] = [gate (F) | up (F)]; block > 0: gu[t] is in groups of `block` gate columns followed by their `block`
     up columns."""
     _dev(gu)
@@ -139,7 +170,7 @@ def silu_mul(gu: torch.Tensor, out: Optional[torch.Tensor] = None, block: int = 
     lib = library("elementwise.cu")
     with region("silu_mul", _nb(gu, out)):
         check(lib.aie_silu_mul(_p(gu), _p(out), c_int(dtype_code(gu)), c_int(T), c_int(F), c_int(block),
-                               c_int(GLU_ACTIVATIONS[activation]), _stream()), "silu_mul")
+                               c_int(GLU_ACTIVATIONS[activation]), *(c_float(v) for v in clamp or _NO_CLAMP), _stream()), "silu_mul")
     return out
 
 
@@ -211,12 +242,21 @@ _TC_SPREAD_KB = 4
 TC_SWIGLU_BLOCK = 64     # gate/up rows per half of a 128-row weight tile
 
 
+def tc_parts(T: int, N: int, K: int, bn: Optional[int] = None, splits: Optional[int] = None) -> int:
+    """The parts that `gemm_tc` cuts K into (`splits` asked for, or its own choice), none of them without K blocks: 64
+    blocks in 9 parts of 8 are 8 parts."""
+    kb = (K + 63) // 64
+    splits = max(1, min(splits or tc_splits(T, N, K, bn or tc_tile(T)), kb))
+    return -(-kb // -(-kb // splits))
+
+
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, err: torch.Tensor,
             bn: Optional[int] = None, splits: Optional[int] = None, swiglu: bool = False,
-            raw_parts: bool = False):
+            raw_parts: bool = False, glu=None, out: Optional[torch.Tensor] = None):
     """bfloat16 x . w^T on tcgen05 tensor cores fed by TMA; None when the sizes are not
     taken (K not a multiple of 8).  swiglu: w is the fused gate/up weight [2F, K] in tiles
-    of 64 gate rows + their 64 up rows; the result is silu(gate) * up, [T, F].
+    of 64 gate rows + their 64 up rows; the result is silu(gate) * up, [T, F], or, with glu = (limit, slope, shift),
+    that of the clamped unit (see silu_mul).  out: float32 [tc_parts(T, N, K), T, N], contiguous, receives the raw parts.
     raw_parts: the parts of a split K are not joined: the result is float32
     [splits, T, N] and whoever reads it adds the parts (the norm and rotary kernels do)."""
     T, K = x.shape
@@ -225,13 +265,14 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, err: torch
         return None
     _dev(x, w, err)
     bn = bn or tc_tile(T)
-    splits = splits or tc_splits(T, N, K, bn)
     if swiglu:
-        splits = 1 if raw_parts else min(splits, 8)
-    kb = (K + 63) // 64
-    splits = max(1, min(splits, kb))
-    splits = -(-kb // -(-kb // splits))      # no part without K blocks: 64 blocks in 9 parts of 8 are 8 parts
-    if raw_parts and splits > 1:
+        splits = 1 if raw_parts else min(splits or tc_splits(T, N, K, bn), 8)
+    splits = tc_parts(T, N, K, bn, splits)
+    if out is not None:
+        if not raw_parts or swiglu or out.shape != (splits, T, N) or out.dtype != torch.float32 or not out.is_contiguous():
+            raise KernelError("gemm_tc: the buffer for the parts does not fit")
+        raw_parts = splits > 1
+    elif raw_parts and splits > 1:
         out = torch.empty((splits, T, N), dtype=torch.float32, device=x.device)
     else:
         raw_parts = False
@@ -241,7 +282,8 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, err: torch
     with region("gemm_tc_swiglu" if swiglu else "gemm_tc", _nb(x, w, out), 2.0 * T * N * K):
         check(lib.aie_gemm_tc(_p(x), _p(w), _p(out), c_int(dtype_code(out)), c_int(T), c_int(N), c_int(K),
                               c_int(out.stride(-2)), c_int(bn), c_int(splits), c_int(1 if swiglu else 0),
-                              c_int(1 if raw_parts else 0), _p(err), _stream()), "gemm_tc")
+                              c_int(1 if raw_parts else 0), *(c_float(v) for v in glu or _NO_CLAMP), _p(err), _stream()),
+              "gemm_tc")
     return out
 
 
@@ -262,13 +304,44 @@ def linear_parts(x: torch.Tensor, w: torch.Tensor, err: Optional[torch.Tensor] =
     return linear(x, w, out_dtype, err)
 
 
+def linear_parts_together(branches, err: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """sum_i x_i . w_i^T for branches (x_i, w_i) whose outputs join the stream together: float32 [parts, T, N], the parts
+    of all products one behind the other, for a consumer that adds them; or the sum [T, N] where a product takes no
+    buffer of ours."""
+    T, N = branches[0][0].shape[0], branches[0][1].shape[0]
+    if err is not None and T <= TC_MAX_TOKENS and all(
+            x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 for x, w in branches):
+        counts = [tc_parts(T, N, x.shape[1]) for x, _ in branches]
+        make = lambda x, w, out: gemm_tc(x, w, torch.float32, err, raw_parts=True, out=out)
+    elif all(x.dtype == torch.float32 for x, _ in branches):
+        counts = [1] * len(branches)
+        make = lambda x, w, out: gemm_f32(x, w, out=out[0])
+    else:
+        ys = [linear(x, w, torch.float32, err) for x, w in branches]
+        y = ys[0]
+        for z in ys[1:]:
+            y = scaled_sum(y, 1.0, z, 1.0)
+        return y
+    buf = torch.empty((sum(counts), T, N), dtype=torch.float32, device=branches[0][0].device)
+    at = 0
+    for (x, w), n in zip(branches, counts):
+        make(x, w, buf[at:at + n])
+        at += n
+    return buf
+
+
+def linear_adds(stream: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether `linear_add` takes this step."""
+    return not (x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or stream.dtype != torch.float32
+                or x.shape[0] <= TC_MAX_TOKENS or stream.shape != (x.shape[0], w.shape[0]) or not stream.is_contiguous())
+
+
 def linear_add(stream: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> bool:
     """stream [T, N] float32 += x . w^T in place, the sum taken in float32 inside the library product (its
     epilogue reads the stream and writes it back), for bfloat16 steps of more than 64 tokens: the branch
     output never travels through memory on its own.  False when the step is not of that kind (nothing
     was done): the caller takes `linear_parts` and lets the next norm add."""
-    if (x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or stream.dtype != torch.float32
-            or x.shape[0] <= TC_MAX_TOKENS or stream.shape != (x.shape[0], w.shape[0]) or not stream.is_contiguous()):
+    if not linear_adds(stream, x, w):
         return False
     _dev(x, w, stream)
     with region("gemm_library", _nb(x, w) + 2 * _nb(stream), 2.0 * x.shape[0] * w.shape[0] * w.shape[1]):
@@ -300,17 +373,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype] = 
 
 
 def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, block: int = 0,
-                  err: Optional[torch.Tensor] = None, activation: str = "silu") -> torch.Tensor:
+                  err: Optional[torch.Tensor] = None, activation: str = "silu", clamp=None) -> torch.Tensor:
     """silu(x . gate^T) * (x . up^T) for the fused gate/up weight [2F, K]; [T, F] in x's
     dtype.  block == 0: rows [0, F) are gate, [F, 2F) up.  block == 64: tiles of 64 gate
     rows + their 64 up rows, which lets the tcgen05 kernel apply the activation in its
-    epilogue when the step is small."""
+    epilogue when the step is small.  activation and clamp: as in silu_mul."""
     if (block == TC_SWIGLU_BLOCK and x.dtype == torch.bfloat16 and w_gu.dtype == torch.bfloat16
-            and x.shape[0] <= TC_MAX_TOKENS and err is not None and activation == "silu"):
-        y = gemm_tc(x, w_gu, x.dtype, err, swiglu=True)
+            and x.shape[0] <= TC_MAX_TOKENS and err is not None and activation in ("silu", "clamped")):
+        y = gemm_tc(x, w_gu, x.dtype, err, swiglu=True, glu=clamp)
         if y is not None:
             return y
-    return silu_mul(linear(x, w_gu, x.dtype, err), block=block, activation=activation)
+    return silu_mul(linear(x, w_gu, x.dtype, err), block=block, activation=activation, clamp=clamp)
 
 
 def linear_rope_kv(x: torch.Tensor, w_qkv: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor,
@@ -1164,29 +1237,45 @@ def sink_attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], pages: t
     return q, gate
 
 
-SINK_FAST_SIZES = (32, 64, 128)      # key and value sizes of the tensor-core kernels of sink_attention
-SINK_FAST_ROWS = (32, 64, 128, 256)  # all keys of a cache row (maps * key size) that the split-KV kernel takes
+SINK_FAST_SIZES = (32, 64, 128)      # key and value sizes that the tensor-core kernels of sink_attention are compiled for
+SINK_FAST_ROWS = (32, 64, 128, 256)  # all keys of a cache row (maps * key size) that the split-KV kernel is compiled for
+
+
+def sink_attention_fast(d: int, e: int, maps: int = 1) -> bool:
+    """Whether the tensor-core kernels take keys of d and values of e elements: steps of 8 up to 128 (smaller sizes are
+    filled up with zeros in shared memory); with several maps the compiled sizes only."""
+    if maps == 1:
+        return d % 8 == 0 and e % 8 == 0 and 0 < d <= 128 and 0 < e <= 128
+    return d in SINK_FAST_SIZES and e in SINK_FAST_SIZES and maps * d in SINK_FAST_ROWS
 
 
 def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Tensor], temp: Optional[torch.Tensor],
                    slope: Optional[torch.Tensor], sink: Optional[torch.Tensor], ctx, work, block_table: torch.Tensor,
                    e: int, scale: float, window: int, keep_first: int, chunk: int = 0, maps: int = 1,
-                   out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+                   out_dtype: Optional[torch.dtype] = None, softcap: float = 0.0, tied: bool = False,
+                   gate_logits: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of a step's query tokens over cache rows [k (d) | v (e)]:
     s(i, j) = (q_i . k_j) * scale * temp[h] - slope[h] * (i - j) over the keys j <= i with i - j < window or
     j < keep_first (window 0: all); softmax whose denominator also holds exp(sink[h]); times gate[i, h].
     q [T, H, d]; gate [T, H], temp, slope, sink [H] float32 or None.  Returns [T, H, e] in q's dtype or `out_dtype`
     (float32).  chunk > 0 (without a window): a query reads the keys of its own chunk of that many positions only.
     maps > 1: rows are [k_0 .. k_(maps-1) | v] and query head h (H counts the heads of all maps) reads key h % maps.
-    bfloat16 with key and value sizes of 32, 64 or 128: lone tokens take the split-KV kernel, portions of prompts
+    softcap c > 0: the scaled product is replaced by c * tanh(it / c).  gate_logits: a float32 view [T, H * e] with any
+    row stride; every output element is multiplied by its sigmoid.  tied: values are the keys, a row is that one vector.
+    bfloat16 with the sizes of `sink_attention_fast`: lone tokens take the split-KV kernel, portions of prompts
     the tiled tensor-core kernel (`work`: the attention work lists); everything else takes the plain kernel."""
     _dev(q, pages, gate, temp, slope, sink, block_table)
     T, H, d = q.shape
     G = pages.shape[1]
     out_dtype = out_dtype or q.dtype
-    if (pages.shape[3] != maps * d + e or H % (G * maps) or pages.dtype != q.dtype or out_dtype not in (q.dtype, torch.float32)
+    w = maps * d + (0 if tied else e)
+    if (pages.shape[3] != w or (tied and (d != e or maps != 1)) or H % (G * maps) or pages.dtype != q.dtype or out_dtype not in (q.dtype, torch.float32)
             or (chunk and (window or keep_first))):
         raise KernelError("sink_attention: shapes, dtypes or masks do not fit")
+    if gate_logits is not None and (gate_logits.dtype != torch.float32 or gate_logits.shape != (T, H * e) or gate_logits.stride(1) != 1):
+        raise KernelError("sink_attention: the gate's logits are a float32 view [T, H * e]")
+    extras = (c_float(softcap), c_int(1 if tied else 0), _p(gate_logits),
+              c_int(gate_logits.stride(0) if gate_logits is not None else 0))
     out = torch.empty((T, H, e), dtype=out_dtype, device=q.device)
     out32 = out if out_dtype == torch.float32 else None
     cost = (0.0, 0.0)
@@ -1199,9 +1288,9 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
         if chunk > 0:
             pairs = [sum(p % chunk + 1 for p in range(int(c), int(c + n))) for n, c in zip(ql, cl)]
             seen, rows = np.asarray(pairs, dtype=float) / ql, cl + ql - cl // chunk * chunk
-        cost = (float(rows.sum()) * G * (maps * d + e) * pages.element_size() + _nb(q, out),
+        cost = (float(rows.sum()) * G * w * pages.element_size() + _nb(q, out, gate_logits),
                 2.0 * float((ql * seen).sum()) * H * (d + e))
-    if q.dtype == torch.bfloat16 and d in SINK_FAST_SIZES and e in SINK_FAST_SIZES and maps * d in SINK_FAST_ROWS:
+    if q.dtype == torch.bfloat16 and sink_attention_fast(d, e, maps):
         fast = library("sink_attention_tc.cu")
         common = (_p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[0]), c_int(pages.shape[2]),
                   c_int(H), c_int(G), c_int(d), c_int(e), c_int(window), c_int(keep_first), c_int(chunk), c_int(maps),
@@ -1221,14 +1310,14 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
                 check(fast.aie_sink_attention_decode(_p(q), _p(pages), _p(out), _p(part_o), _p(part_lse), _p(gate),
                                                      _p(temp), _p(slope), _p(sink), _p(work.decode_tokens), c_int(n),
                                                      _p(ctx.positions), _p(ctx.token_req), *common, c_int(S),
-                                                     _p(out32), _p(ctx.err), _stream()), "sink_attention_decode")
+                                                     *extras, _p(out32), _p(ctx.err), _stream()), "sink_attention_decode")
         if work.n_decode < ctx.R:
             tiles = work.prefill_tiles
             share = 1.0 - float(work.n_decode) / T
             with region("sink_attention_prefill", cost[0] * share, cost[1] * share):
                 check(fast.aie_sink_attention_prefill(_p(q), _p(pages), _p(out), _p(gate), _p(temp), _p(slope), _p(sink),
                                                       _p(tiles), c_int(tiles.shape[0]), _p(ctx.q_start), _p(ctx.q_len),
-                                                      _p(ctx.ctx_len), *common, _p(out32), _p(ctx.err), _stream()),
+                                                      _p(ctx.ctx_len), *common, *extras, _p(out32), _p(ctx.err), _stream()),
                       "sink_attention_prefill")
         return out
     lib = library("sink_attention.cu")
@@ -1237,7 +1326,7 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
                                            _p(temp), _p(slope), _p(sink), _p(ctx.positions), _p(ctx.token_req), _p(block_table),
                                            c_int(block_table.shape[1]), c_int(pages.shape[0]), c_int(pages.shape[2]),
                                            c_int(T), c_int(H), c_int(G), c_int(d), c_int(e), c_int(window),
-                                           c_int(keep_first), c_int(chunk), c_int(maps), c_float(scale), _p(None),
+                                           c_int(keep_first), c_int(chunk), c_int(maps), c_float(scale), *extras, _p(None),
                                            _p(ctx.err), _stream()),
               "sink_attention_plain")
     return out
@@ -1391,7 +1480,8 @@ def normed_attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_weig
                         k_weight: Optional[torch.Tensor], eps: float, inv_freq: Optional[torch.Tensor], rot_dims: int,
                         halves: bool, pages: torch.Tensor, ctx, block_table: torch.Tensor, H: int, G: int, d: int, e: int,
                         mix_from: Optional[torch.Tensor] = None, mix_lambda: Optional[torch.Tensor] = None,
-                        keep_values: bool = False, write: bool = True, maps: int = 1, per_head: bool = False):
+                        keep_values: bool = False, write: bool = True, maps: int = 1, per_head: bool = False,
+                        magnitude: float = 1.0, unit: bool = False, tied: bool = False):
     """From a step's fused projection whose first columns are [q (H d) | k (G d) | v (G e)] (float32 [T, >= that]):
     biases added; all of q divided by its root mean square over the H d elements, times q_weight (k likewise; None: no
     norm); the first rot_dims elements of every head of q and k rotated by the token's position (pairs of neighbours,
@@ -1399,22 +1489,27 @@ def normed_attn_prepare(proj: torch.Tensor, bias: Optional[torch.Tensor], q_weig
     the device).  q [T, H, d] in the cache's dtype is returned; with `write`, the token's cache row [k | v] is
     written.  keep_values: the values as they are cached are also returned in float32 [T, G e].
     pages [num_pages, G, P, d + e].  per_head: every head of q and of k is normed by itself, with weights [d].
-    maps > 1: k has G * maps heads, a row is [k_0 .. k_(maps-1) | v], and H counts the query heads of all maps."""
+    maps > 1: k has G * maps heads, a row is [k_0 .. k_(maps-1) | v], and H counts the query heads of all maps.
+    magnitude multiplies the rotated elements; unit: every head of q and k is divided by its root mean square behind the
+    rotation (both with neighbouring pairs, without a norm over the whole projection and without mixing).  tied: there are
+    no columns of v, and a cache row is the key alone."""
     _dev(proj, bias, q_weight, k_weight, inv_freq, pages, block_table, mix_from, mix_lambda)
     T, ld = proj.shape
-    n = H * d + G * (maps * d + e)
+    w = maps * d + (0 if tied else e)
+    n = H * d + G * w
     nq, nk = (d, d) if per_head else (H * d, G * maps * d)
-    if (proj.dtype != torch.float32 or ld < n or pages.shape[1] != G or pages.shape[3] != maps * d + e
-            or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != n))
+    if (proj.dtype != torch.float32 or ld < n or pages.shape[1] != G or pages.shape[3] != w
+            or (tied and (keep_values or mix_from is not None)) or (bias is not None and (bias.dtype != torch.float32 or bias.numel() != n))
             or (q_weight is not None and (k_weight is None or q_weight.numel() != nq or k_weight.numel() != nk))
             or (mix_from is not None and (mix_from.dtype != torch.float32 or mix_from.shape != (T, G * e) or mix_lambda is None))):
         raise KernelError("normed_attn_prepare: shapes or dtypes do not fit")
     q = torch.empty((T, H, d), dtype=pages.dtype, device=proj.device)
     kept = torch.empty((T, G * e), dtype=torch.float32, device=proj.device) if keep_values else None
     lib = library("sink_attention.cu")
-    with region("normed_attn_prepare", T * n * 4 + _nb(q, kept, mix_from) + T * G * (maps * d + e) * pages.element_size()):
+    with region("normed_attn_prepare", T * n * 4 + _nb(q, kept, mix_from) + T * G * w * pages.element_size()):
         check(lib.aie_normed_attn_prepare(_p(proj), c_int(ld), _p(bias), _p(q_weight), _p(k_weight), c_float(eps),
-                                          _p(inv_freq), c_int(rot_dims), c_int(1 if halves else 0), _p(mix_from),
+                                          _p(inv_freq), c_int(rot_dims), c_int(1 if halves else 0), c_float(magnitude),
+                                                  c_int(1 if unit else 0), c_int(1 if tied else 0), _p(mix_from),
                                           _p(mix_lambda), _p(kept), _p(q), _p(pages), c_int(dtype_code(pages)),
                                           _p(ctx.positions), _p(ctx.token_req), _p(block_table), c_int(block_table.shape[1]),
                                           c_int(pages.shape[0]), c_int(pages.shape[2]), c_int(T), c_int(H), c_int(G), c_int(d),

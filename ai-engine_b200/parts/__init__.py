@@ -1,7 +1,8 @@
 from .attention import ATTENTION_WORK, AttentionWork, GQAAttention
 from .base import (Block, BuildEnv, CacheNeed, FeedForward, KVRequest, LayerCache, Mixer, Norm, Part,
                    PositionEncoding, StateRequest, StepPlanner, TokenFilter)
-from .block import DepthAveragedBlock, GatedPostNormBlock, ParallelBlock, PreNormBlock, SandwichNormBlock
+from .block import (DepthAveragedBlock, GatedPostNormBlock, ParallelBlock, PreNormBlock, SandwichNormBlock,
+                    TwoNormParallelBlock)
 from .conv import CausalShortConv
 from .embedding import LMHead, TokenEmbedding
 from .latent_attention import LATENT_WORK, LatentAttention, LatentWork
@@ -53,6 +54,7 @@ register("mixer", "differential_attention", DifferentialAttention)
 register("filter", "token_shift", TokenShift)
 register("feed_forward", "token_side", TokenSide)
 register("block", "gated_post_norm", GatedPostNormBlock)
+register("block", "parallel_two_norms", TwoNormParallelBlock)
 
 __all__ = ["ATTENTION_WORK", "AttentionWork", "GQAAttention", "Block", "BuildEnv", "CacheNeed", "FeedForward",
            "KVRequest", "LayerCache", "Mixer", "Norm", "Part", "PositionEncoding", "StateRequest", "StepPlanner", "PreNormBlock", "LMHead",
@@ -63,4 +65,4 @@ __all__ = ["ATTENTION_WORK", "AttentionWork", "GQAAttention", "Block", "BuildEnv
            "LatentAttention", "DecayLinearAttention", "PolyNormFF", "TableMoE", "SandwichNormBlock", "ParallelMixers",
            "ScalarDecayStateSpace", "RoutedMoE", "SinkWindowAttention", "GatedDeltaRule", "DenseFF", "SinusoidalPositions",
            "DynamicTanh", "ParallelBlock", "ForgetGateLinearAttention", "NormedGatedAttention", "DifferentialAttention", "TokenShift", "TokenSide",
-           "GatedPostNormBlock", "rotary_magnitude"]
+           "GatedPostNormBlock", "TwoNormParallelBlock", "rotary_magnitude"]

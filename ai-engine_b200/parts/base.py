@@ -155,6 +155,9 @@ class Mixer(Part):
     # True: forward takes `add_to=stream` (the float32 residual stream) and may add its output there itself,
     # returning None instead of the output (a block then hands no pending branch to the next norm)
     adds_in_place = False
+    # True: forward takes `leave_projection=True`, with which it returns (a, w): its output is a . w^T, a product that the
+    # caller makes (with another branch's, or into the stream)
+    leaves_projection = False
     # True: the output projection has a bias, kept as `output_bias` (float32 [hidden]); forward takes `leave_bias=True`,
     # with which the caller adds it itself
     leaves_bias = False
@@ -167,6 +170,7 @@ class FeedForward(Part):
     """Token-local: forward(h [T, hidden], ctx) -> [T, hidden], float32 or the compute dtype."""
 
     adds_in_place = False      # as for a Mixer
+    leaves_projection = False  # as for a Mixer
     # True: forward takes `leave_rows=True`, with which it returns ops.ExpertRows (a token's expert rows and their
     # weights) for a caller that sums them itself, and `logits=` (float32 [(parts,) T, n]) for the product of its
     # input with the weight that `router_weight()` hands out, when the caller has made it along with one of its own
@@ -191,6 +195,11 @@ class Norm(Part):
 
     def forward(self, x, delta=None, rows=None, write_back=True) -> torch.Tensor:
         raise NotImplementedError
+
+    def pairs_with(self, other) -> bool:
+        """Whether `forward_pair(other, ...)` can make this norm's output and that of `other` (a norm, or None for no
+        second output) in one pass over a row."""
+        return False
 
 
 class PositionEncoding(Part):

@@ -33,7 +33,7 @@ class PreNormBlock(Block):
             raise ValueError("pre-norm block: a feed-forward comes with its norm")
         self.hidden = env.hidden_size
         self.w_mix = None
-        self.needs_embedding_output = "input_mix" in spec.tensors
+        self.needs_embedding_output = self.replaces_stream = "input_mix" in spec.tensors
 
     def tensor_specs(self):
         name = self.spec.tensors.get("input_mix")
@@ -230,6 +230,64 @@ class ParallelBlock(Block):
         if made is not None:
             ctx.normed_ahead = (nxt, made)
         return x, None
+
+
+class TwoNormParallelBlock(Block):
+    """A block whose mixer and feed-forward read the same stream, each behind a norm of its own, and are added together:
+
+        x = x + (mixer(mixer_norm(x)) + ffn(ffn_norm(x)))
+
+    The feed-forward with its norm is optional.  With the tensor `pass_steps` [passes, hidden] the layer opens a pass over
+    a group of layers that runs several times (params: passes): what it reads, and what its branches are added to, is
+
+        x + steps[0] in the first pass,     (x + x0) + steps[t] in pass t > 0,     x0 the embedding's output
+
+    with t = ctx.pass_index.  One kernel adds what the branches before left, opens the pass and makes both norms' outputs
+    (a row has one root mean square).  Where both branches can leave their last product to the block, the two products
+    of a small step write their parts side by side into one buffer, which is the next norm's pending branch; in larger
+    steps both add to the stream in place."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "ffn_norm": "norm", "ffn": "feed_forward"}
+    optional_roles = ("ffn_norm", "ffn")
+
+    def __init__(self, spec, env, parts):
+        super().__init__(spec, env)
+        self.mixer_norm, self.mixer = parts["mixer_norm"], parts["mixer"]
+        self.ffn_norm, self.ffn = parts.get("ffn_norm"), parts.get("ffn")
+        if (self.ffn is None) != (self.ffn_norm is None):
+            raise ValueError("two-norm block: a feed-forward comes with its norm")
+        if not self.mixer_norm.pairs_with(self.ffn_norm):
+            raise ValueError("two-norm block: both norms divide by the same root mean square")
+        for part in (self.mixer, self.ffn):
+            if part is not None and not part.leaves_projection:
+                raise ValueError("two-norm block: both branches leave their last product to the block")
+        self.hidden = env.hidden_size
+        self.needs_embedding_output = "pass_steps" in spec.tensors and int(spec.params["passes"]) > 1
+        self.steps = None
+
+    def tensor_specs(self):
+        name = self.spec.tensors.get("pass_steps")
+        return [TensorSpec(name, (int(self.spec.params["passes"]), self.hidden), std=0.5)] if name else []
+
+    def load(self, source):
+        name = self.spec.tensors.get("pass_steps")
+        if name:
+            self.steps = source.get(name).float().contiguous()
+
+    def forward(self, x, pending, ctx, caches):
+        step = extra = None
+        if self.steps is not None:
+            step = self.steps[ctx.pass_index]
+            extra = ctx.embedding_output if ctx.pass_index > 0 else None
+        h, h2 = self.mixer_norm.forward_pair(self.ffn_norm, x, pending, extra, step)
+        branches = [self.mixer.forward(h, ctx, caches.get("mixer"), leave_projection=True)]
+        if self.ffn is not None:
+            branches.append(self.ffn.forward(h2, ctx, leave_projection=True))
+        if all(ops.linear_adds(x, a, w) for a, w in branches):
+            for a, w in branches:
+                ops.linear_add(x, a, w)
+            return x, None
+        return x, ops.linear_parts_together(branches, ctx.err)
 
 
 class GatedPostNormBlock(Block):

@@ -11,8 +11,11 @@ from .base import FeedForward
 
 class SwiGLU(FeedForward):
     """params: hidden_size, intermediate_size, activation (default "silu"; "relu" and "gelu_tanh" give
-    down(act(gate(x)) * up(x)) with that act).  tensors: gate, up [F, hidden], down [hidden, F].  gate and up
-    are fused into one [2F, hidden] weight at load."""
+    down(act(gate(x)) * up(x)) with that act; "clamped", with limit, slope and shift, gives
+    down(g * sigmoid(slope * g) * (u + shift)) with g = min(gate(x), limit) and u = up(x) kept within +-limit).
+    tensors: gate, up [F, hidden], down [hidden, F].  gate and up are fused into one [2F, hidden] weight at load."""
+
+    leaves_projection = True
 
     def __init__(self, spec, env):
         super().__init__(spec, env)
@@ -22,6 +25,12 @@ class SwiGLU(FeedForward):
         if self.activation not in ops.GLU_ACTIVATIONS:
             raise ValueError(f"gated feed-forward: activation `{self.activation}` is not known "
                              f"({', '.join(ops.GLU_ACTIVATIONS)})")
+        self.clamp = None
+        if self.activation == "clamped":
+            p = spec.params
+            self.clamp = (float(p.get("limit", float("inf"))), float(p.get("slope", 1.0)), float(p.get("shift", 0.0)))
+            if not self.clamp[0] > 0:
+                raise ValueError(f"gated feed-forward: limit must be positive, got {self.clamp[0]}")
         self.w_gu = self.w_down = None
         self.block = 0
 
@@ -38,7 +47,7 @@ class SwiGLU(FeedForward):
         # bfloat16: 64 gate rows then their 64 up rows, tile by tile, so that a 128-row
         # weight tile of the tensor-core kernel holds both halves of 64 outputs
         self.block = ops.TC_SWIGLU_BLOCK if (dt == torch.bfloat16 and self.inter % ops.TC_SWIGLU_BLOCK == 0
-                                             and self.activation == "silu") else 0
+                                             and self.activation in ("silu", "clamped")) else 0
         if self.block:
             b = self.block
             self.w_gu = torch.stack([g.view(-1, b, self.hidden), u.view(-1, b, self.hidden)], dim=1) \
@@ -55,9 +64,11 @@ class SwiGLU(FeedForward):
 
     adds_in_place = True
 
-    def forward(self, h, ctx, add_to=None):
+    def forward(self, h, ctx, add_to=None, leave_projection=False):
         err = ctx.err if ctx is not None else None
-        a = ops.linear_swiglu(h, self.w_gu, self.block, err, self.activation)
+        a = ops.linear_swiglu(h, self.w_gu, self.block, err, self.activation, self.clamp)
+        if leave_projection:
+            return a, self.w_down
         if add_to is not None and ops.linear_add(add_to, a, self.w_down):
             return None
         return ops.linear_parts(a, self.w_down, err)   # joins the residual in float32, inside the next norm

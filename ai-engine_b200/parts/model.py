@@ -171,11 +171,12 @@ class Model:
             pe.add_to(x, ctx)
         if self.keeps_embedding_output:
             # a block that reads the embedding's output later finds it on the step; layers before it write into the
-            # stream in place, so it is copied unless that block comes first and makes a stream of its own
+            # stream in place, so it is copied unless the first block makes a stream of its own
             first = self.layers[self.order[0].layer].block
-            ctx.embedding_output = x if getattr(first, "needs_embedding_output", False) else x.clone()
+            ctx.embedding_output = x if getattr(first, "replaces_stream", False) else x.clone()
         pending = None
         for i, rs in enumerate(self.order):
+            ctx.pass_index = rs.pass_index
             x, pending = self.layers[rs.layer].block.forward(x, pending, ctx, cache.layer_cache(i, ctx))
             if streams is not None:
                 full = x.clone()

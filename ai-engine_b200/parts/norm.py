@@ -38,6 +38,18 @@ class RMSNorm(Norm):
         return ops.add_rmsnorm(x, delta, self.weight, self.eps, self.out_dtype, rows=rows,
                                write_back=write_back)
 
+    def pairs_with(self, other) -> bool:
+        """Whether this norm and `other` differ in their weights only, so that one pass over a row makes both outputs (None: there is
+        no second one)."""
+        return other is None or (isinstance(other, RMSNorm) and (other.size, other.eps, other.out_dtype)
+                == (self.size, self.eps, self.out_dtype))
+
+    def forward_pair(self, other, x, delta=None, extra=None, step=None):
+        """s = x (+ delta) (+ extra) (+ step, one row for all tokens), stored into the float32 stream x; returns this
+        norm's output of s and that of `other` (None: no second output, None is returned for it)."""
+        w2 = other.weight if other is not None else None
+        return ops.add_rmsnorm_pair(x, delta, self.weight, w2, self.eps, self.out_dtype, extra=extra, step=step)
+
     def add_normed(self, x, y, **options):
         """x += norm(y) in place, for a norm on a sublayer's output; the options (a gate on y, a bias, the new stream in
         a compute dtype, ...) and the result are those of `ops.gated_norm_add`."""

@@ -34,9 +34,12 @@ class LayerSpec:
 class RunStep:
     """One entry of the run order.  `layer` indexes `ModelSpec.layers` (a layer may
     be named by several entries).  `cache_from`: the index of an earlier entry
-    whose cache this one reads without writing; None: a cache of its own."""
+    whose cache this one reads without writing; None: a cache of its own.  `pass_index`: the
+    how-manieth run of a group of layers that runs several times this entry belongs to (a block reads it
+    as `ctx.pass_index`)."""
     layer: int
     cache_from: Optional[int] = None
+    pass_index: int = 0
 
 
 @dataclass
