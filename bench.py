@@ -149,6 +149,25 @@ def vatazen_shape(width, layers=8):
                 token_side=dict(dim=width // 16), layers=[dict((lat, att)[i % 2], mlp=moe) for i in range(layers)])
 
 
+def kagatar_shape(width, layers=8):
+    """A Kagatar configuration with layers of the sizes real models of its kind have: heads of 128 for keys and values (a
+    quarter of them key/value heads); windows of 1,024 keys where the values are the keys and where the scores are
+    bounded, all keys in the gated layers; half of a gated head and the whole of a bounded one rotated, positions
+    stretched by 8; a clamped feed-forward of 3 x width.  The pattern (tied, gated, bounded) repeats; the first three
+    layers run twice, so `layers` layer runs hold layers - 3 layers."""
+    H = width // 128
+    mix = lambda **more: dict(heads=H, kv_heads=max(1, H // 4), dim=128, vdim=128, scale=128 ** -0.5, **more)
+    tied = dict(type="attention", mixer=mix(mask=dict(size=1024)))
+    gated = dict(type="attention_2", mixer=mix(rot=dict(base=500000.0, dims=64, scaling=dict(
+        factor=8.0, original=4096, fast=32.0, slow=1.0))))
+    capped = dict(type="attention_3", mixer=mix(mask=dict(size=1024), softcap=30.0, rot=dict(base=500000.0, dims=128, scaling=dict(
+        factor=8.0, low=1.0, high=4.0, original=4096))))
+    n = max(3, layers - 3)
+    return dict(architecture="Kagatar", vocab=32000, width=width, norm=dict(eps=1e-5), embedding=dict(scale=1.0),
+                logit_softcap=30.0, loop=dict(start=0, stop=3, times=2),
+                layers=[dict((tied, gated, capped)[i % 3], mlp=dict(kind="dense", ff=3 * width, limit=7.0)) for i in range(n)])
+
+
 def llama_like(width, layers=8):
     """The closest existing model at equal size: the same width, layers, heads of 128 (a quarter of them kv heads)
     and a feed-forward of 3 x width, which is what a Pifutar token uses (4 experts of width / 2 + the shared one)."""
@@ -691,10 +710,10 @@ def main():
                     help="time one part only and print its numbers (for profiling)")
     ap.add_argument("--profile", action="store_true",
                     help="CUDA-event time, bytes, flops and roofline fraction per class of kernel (eager launches)")
-    ap.add_argument("--shape", choices=["8b", "1b", "3b"] + [f"{m}-{w}" for m in ("pifutar", "zupitar", "tizodra", "fokisun", "vatazen", "llama") for w in WIDTHS],
+    ap.add_argument("--shape", choices=["8b", "1b", "3b"] + [f"{m}-{w}" for m in ("pifutar", "zupitar", "tizodra", "fokisun", "vatazen", "kagatar", "llama") for w in WIDTHS],
                     default="8b",
                     help="layer sizes for --profile and --only decode|prefill (the headline run is always the 8B shape); "
-                         "pifutar-1k|2k|4k, zupitar-1k|2k|4k, tizodra-1k|2k|4k, fokisun-1k|2k|4k, vatazen-1k|2k|4k: those designs at that width, llama-1k|2k|4k: Llama at equal size beside them "
+                         "pifutar-1k|2k|4k, zupitar-1k|2k|4k, tizodra-1k|2k|4k, fokisun-1k|2k|4k, vatazen-1k|2k|4k, kagatar-1k|2k|4k: those designs at that width, llama-1k|2k|4k: Llama at equal size beside them "
                          "(8 layers unless --layers says otherwise)")
     ap.add_argument("--prompt-len", type=int, default=PROMPT_LEN, help="cached tokens per request for --profile / --only decode")
     ap.add_argument("--skip-workloads", action="store_true", help="leave the 1B and 3B serving workloads out of `points`")
@@ -741,7 +760,7 @@ def main():
     if "-" in a.shape and (a.profile or a.only):
         family, w = a.shape.split("-")
         layers = a.layers if a.layers != LLAMA3_8B["num_hidden_layers"] else 8
-        cfg = dict(pifutar=pifutar_shape, zupitar=zupitar_shape, tizodra=tizodra_shape, fokisun=fokisun_shape, vatazen=vatazen_shape, llama=llama_like)[family](WIDTHS[w], layers)
+        cfg = dict(pifutar=pifutar_shape, zupitar=zupitar_shape, tizodra=tizodra_shape, fokisun=fokisun_shape, vatazen=vatazen_shape, kagatar=kagatar_shape, llama=llama_like)[family](WIDTHS[w], layers)
     else:
         cfg = dict({"8b": LLAMA3_8B, "1b": LLAMA32_1B, "3b": LLAMA32_3B}.get(a.shape, LLAMA3_8B) if (a.profile or a.only) else LLAMA3_8B)
         if a.layers != LLAMA3_8B["num_hidden_layers"] or a.shape == "8b":

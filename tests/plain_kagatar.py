@@ -74,13 +74,11 @@ def rotate_neighbours(x: torch.Tensor, positions, freqs: List[float], magnitude:
     """x [T, heads, d]: elements 2i and 2i + 1 of every head turned by position * freqs[i], the turned ones scaled by
     `magnitude`; what lies behind the last pair stays."""
     y = x.clone()
-    for t in range(x.shape[0]):
-        for i, f in enumerate(freqs):
-            a = float(positions[t]) * f
-            c, s = math.cos(a) * magnitude, math.sin(a) * magnitude
-            u, v = x[t, :, 2 * i], x[t, :, 2 * i + 1]
-            y[t, :, 2 * i] = u * c - v * s
-            y[t, :, 2 * i + 1] = v * c + u * s
+    p = torch.tensor([float(t) for t in positions], dtype=torch.float64)
+    for i, f in enumerate(freqs):
+        c, s = ((fn(p * f) * magnitude).to(x.dtype)[:, None] for fn in (torch.cos, torch.sin))
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        y[..., 2 * i], y[..., 2 * i + 1] = u * c - v * s, v * c + u * s
     return y
 
 
@@ -99,15 +97,13 @@ def softmax_over_sight(q, k, v, scale: float, size: int, cap: Optional[float] = 
     """q [T, H, d], k [T, G, d], v [T, G, e] of one sequence -> [T, H, e]: the token at place i reads the places
     first_key(i) .. i; head h reads key/value head h // (H / G)."""
     T, H = q.shape[:2]
-    G = k.shape[1]
+    k, v = (t.repeat_interleave(H // t.shape[1], dim=1) for t in (k, v))       # one key/value head per query head
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
     for i in range(T):
-        j0 = first_key(i, size)
-        for h in range(H):
-            g = h // (H // G)
-            s = bounded((k[j0:i + 1, g] @ q[i, h]) * scale, cap)
-            p = torch.exp(s - s.max())
-            out[i, h] = (p[:, None] * v[j0:i + 1, g]).sum(dim=0) / p.sum()
+        seen = slice(first_key(i, size), i + 1)
+        s = bounded((k[seen] * q[i]).sum(dim=-1) * scale, cap)                 # [keys seen, H]
+        p = torch.exp(s - s.max(dim=0).values)
+        out[i] = (p[..., None] * v[seen]).sum(dim=0) / p.sum(dim=0)[:, None]
     return out
 
 
@@ -183,7 +179,8 @@ def layer_update(x, L: dict, w: Dict[str, torch.Tensor], eps: float, positions):
     """mixer(norm1(x)) + ff(norm2(x)), both of the same x."""
     y = MIXERS[L["type"]](rms(x, eps) * w["norm1"], sub(w, "mix."), L["mixer"], eps, positions)
     if L.get("mlp"):
-        y = y + clamped_ff(rms(x, eps) * w["norm2"], w["mlp.gate"], w["mlp.up"], w["mlp.down"], L["mlp"]["limit"])
+        y = y + clamped_ff(rms(x, eps) * w["norm2"], w["mlp.gate"], w["mlp.up"], w["mlp.down"],
+                           L["mlp"].get("limit", math.inf))
     return y
 
 
