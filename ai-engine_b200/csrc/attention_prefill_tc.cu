@@ -27,6 +27,11 @@
 //                      (in units of log2 e): P stays below 2^8 and the row of O in tensor memory is
 //                      rescaled on few tiles; the final division by the running sum makes the
 //                      result the same softmax.
+// The extended form (EXT) of this kernel adds, for layers that want them: a window (key tiles before it are never
+// loaded, nor are pages that the window has passed), scores kept within +-cap by a tanh, probabilities that enter the
+// product with the values as two bfloat16 terms (the rounded one over the first half of the scores' columns, what
+// rounding left over the second: 16 bits of mantissa), a sigmoid gate on every output element, and cache rows
+// [k | v] or, with the values being the keys, [k] of one plane.
 // The value rows of keys past the sequence's last token are zeroed in shared memory before the
 // last tile's P . V, so a probability of 0 never meets what an unwritten cache slot holds.
 // The softmax warps hand a tile's probabilities to the issuing warp at a named hardware barrier (bar.arrive /
@@ -57,6 +62,29 @@ template <int HD> struct AtSmem {
     static constexpr int q_off = 1024, k_off = q_off + tile, v_off = k_off + NST * tile, end = v_off + NST * tile;
     static constexpr int bytes = 1024 + end;
 };
+
+// what the extended form of the kernel takes beside the plain one's arguments
+struct AtExt {
+    int window;                   // 0: every earlier key
+    float cap;                    // 0: scores are not bounded
+    const float* gate_logits;     // [T, >= H * HD] float32, rows ld_gate apart, or null
+    int ld_gate;
+};
+
+// tanh(z) for |z| <= 1 as an odd polynomial of degree 15, two at a time (z2 = z^2 and z as packed pairs); the
+// coefficients are a weighted least-squares fit on Chebyshev nodes; relative error in float32 under 2e-7 over the interval
+#define AT_TANH_COEFS \
+    {1.f, -0.333332777f, 0.133321598f, -0.0538709052f, 0.0214648023f, -0.00791741814f, 0.00228221063f, -0.000353340118f}
+__device__ __forceinline__ unsigned long long at_fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+    unsigned long long r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ unsigned long long at_mul2(unsigned long long a, unsigned long long b) {
+    unsigned long long r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
 
 // shared-memory descriptor of an MN-major operand: rows of 64 elements (128 bytes) along MN,
 // groups of 8 K-rows `sbo` bytes apart, blocks of 64 MN elements `lbo` bytes apart
@@ -113,14 +141,14 @@ __device__ __forceinline__ float at_hi(unsigned long long v) {
                    "r"(v[16]), "r"(v[17]), "r"(v[18]), "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]),   \
                    "r"(v[24]), "r"(v[25]), "r"(v[26]), "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31]) : "memory")
 
-template <int HD>
+template <int HD, bool EXT>
 __global__ void __launch_bounds__(AT_THREADS, 1)
 paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                         const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                         const int* __restrict__ tiles, int n_tiles, const int* __restrict__ q_start,
                         const int* __restrict__ q_len, const int* __restrict__ ctx_len,
                         const int* __restrict__ block_table, int bt_width, int num_pages, int P, int H, int K,
-                        float scale, unsigned* err) {
+                        float scale, unsigned* err, const AtExt ext) {
     extern __shared__ unsigned char at_raw[];
     unsigned char* sm = reinterpret_cast<unsigned char*>(((size_t)at_raw + 1023) & ~(size_t)1023);
     unsigned long long* q_full = reinterpret_cast<unsigned long long*>(sm);
@@ -151,7 +179,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const int rows_valid = min(AT_M, q_len[r] - q_off);
     const int p0 = ctx_len[r] + q_off;                 // position of the tile's first query
     const int p_last = p0 + rows_valid - 1;            // and of its last valid one
-    const int n_kt = p_last / AT_N + 1;                // key tiles 0 .. n_kt - 1
+    // first key that any row reads, and the tile it lies in; tile j of the loops below is key tile kt0 + j
+    const int lo_min = EXT && ext.window > 0 ? max(p0 - ext.window + 1, 0) : 0;
+    const int kt0 = lo_min / AT_N;
+    const int n_kt = p_last / AT_N + 1 - kt0;          // key tiles
     const int ppt = AT_N / P;                          // pages per key tile
 
     if (tid == 0) {
@@ -178,6 +209,10 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
     const unsigned tmem_base = *tmem_slot;
+    if (EXT) {
+        pdl_launch_dependents();
+        pdl_wait();
+    }
 
     if (warp == 0) {
             if (lane == 0) {
@@ -190,16 +225,29 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         const int* bt = block_table + (size_t)r * bt_width;
         const int lp = 31 - __clz(P);                      // P is a power of two
         auto page_of = [&](int jj) {
-            const int pidx = jj * ppt + lane;
+            const int pidx = (kt0 + jj) * ppt + lane;
             return (lane < ppt && (pidx << lp) <= p_last && pidx < bt_width) ? bt[pidx] : -1;
         };
         int page = page_of(0);
         bool ok = true;
+        // pages of the first tile that lie wholly before the window: they may be gone, so they are not loaded, and
+        // their value rows are zeroed before the tile's barrier is armed
+        const int skip = EXT ? (lo_min >> lp) - kt0 * ppt : 0;
+        if (EXT && skip > 0) {
+            for (int i = lane; i < skip * P * HV * 8; i += 32) {
+                const int row = i / (HV * 8), c = i % (HV * 8);
+                *reinterpret_cast<uint4*>(v_s + (row >> 3) * GROUP + (c >> 3) * 1024 + (row & 7) * 128 + (c & 7) * 16) =
+                    make_uint4(0, 0, 0, 0);
+            }
+            asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");
+            __syncwarp();
+        }
         for (int j = 0; j < n_kt && ok; ++j) {
             const int st = j % NST;
             const int page_next = j + 1 < n_kt ? page_of(j + 1) : -1;
-            const int n_pages = min(ppt, ((p_last - j * AT_N) >> lp) + 1);      // pages of this tile that hold keys
-            const bool have = lane < n_pages;
+            const int n_pages = min(ppt, ((p_last - (kt0 + j) * AT_N) >> lp) + 1);      // pages of this tile that hold keys
+            const int from = EXT && j == 0 ? skip : 0;
+            const bool have = lane >= from && lane < n_pages;
             const bool valid = have && page >= 0 && page < num_pages;
             if (have && !valid) atomicOr(err, AIE_DEV_PAGE_OOB);
             // a missing page is flagged; page 0 stands in for it so that the byte count of the barrier holds
@@ -208,7 +256,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             if (lane == 0) {
                 const unsigned ph = ((j / NST) & 1) ^ 1;
                 ok = mbar_wait(&k_empty[st], ph, abort_flag, err) && mbar_wait(&v_empty[st], ph, abort_flag, err);
-                if (ok) mbar_expect_tx(&kv_full[st], 2u * (unsigned)n_pages * (unsigned)P * (unsigned)(HD * 2));
+                if (ok) mbar_expect_tx(&kv_full[st], 2u * (unsigned)(n_pages - from) * (unsigned)P * (unsigned)(HD * 2));
             }
             ok = __shfl_sync(0xffffffffu, ok ? 1 : 0, 0) != 0;
             if (!ok) break;
@@ -223,7 +271,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         // the last tile: zero the value rows of keys past the sequence's end (whole warp)
         {
             const int j = n_kt - 1, st = j % NST;
-            const int first_bad = p_last + 1 - j * AT_N;       // rows [first_bad, 128) are not keys
+            const int first_bad = p_last + 1 - (kt0 + j) * AT_N;       // rows [first_bad, 128) are not keys
             bool ok2 = true;
             if (first_bad < AT_N) {
                 if (lane == 0) ok2 = mbar_wait(&kv_full[st], (j / NST) & 1, abort_flag, err);
@@ -301,6 +349,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 for (int ks = 0; ks < 8; ++ks)
                     umma_a_tmem(tmem_base + 256u, tp + (unsigned)(ks * 8), dv + (unsigned long long)((ks * 2 * GROUP) >> 4),
                                 idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
+                if (EXT) {
+#pragma unroll
+                    for (int ks = 0; ks < 8; ++ks)           // what rounding left of the probabilities
+                        umma_a_tmem(tmem_base + 256u, tp + 64u + (unsigned)(ks * 8),
+                                    dv + (unsigned long long)((ks * 2 * GROUP) >> 4), idesc_o, 1u);
+                }
                 umma_commit(&v_empty[st0]);
                 umma_commit(o_done);
             }
@@ -312,7 +366,12 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
         const int qpos = p0 + row;
         const unsigned lane_addr = (unsigned)(quarter * 32) << 16;
         const unsigned tmem_o = tmem_base + 256u;
-        const float sl2 = scale * 1.4426950408889634f;      // scores in units of log2(e): exp2 below
+        const float log2e = 1.4426950408889634f;
+        const bool capped = EXT && ext.cap > 0.f;
+        const float sl2 = capped ? ext.cap * log2e : scale * log2e;      // scores in units of log2(e): exp2 below
+        const float z_of = capped ? scale / ext.cap : 0.f;
+        const int low = EXT && ext.window > 0 ? qpos - ext.window + 1 : 0;      // first key this row reads
+        const int low_last = EXT && ext.window > 0 ? p_last - ext.window + 1 : 0;
         float m_run = -INFINITY, l_run = 0.f;
         bool ok = true;
         for (int j = 0; j < n_kt; ++j) {
@@ -328,7 +387,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 continue;
             }
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
-            const int kbase = j * AT_N;
+            const int kbase = (kt0 + j) * AT_N;
             const bool edge = kbase + AT_N - 1 > p0;     // the tile touches the diagonal or the sequence's end
             // the row of scores in registers (all four loads in flight at once), masked; its maximum
             unsigned sv[128];
@@ -337,10 +396,46 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             AT_LD32((sv + 64), tmem_s + lane_addr + 64);
             AT_LD32((sv + 96), tmem_s + lane_addr + 96);
             asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+            if (capped) {
+                // s <- tanh(s scale / cap), times cap where the exponent is made
+                float big = 0.f;
+#pragma unroll
+                for (int i = 0; i < 128; i += 2)
+                    big = at_max3(big, fabsf(__uint_as_float(sv[i])), fabsf(__uint_as_float(sv[i + 1])));
+                if (__all_sync(0xffffffffu, big * z_of <= 1.f)) {
+                    constexpr float tc[8] = AT_TANH_COEFS;
+                    const unsigned long long zz = at_pack2(z_of, z_of);
+#pragma unroll
+                    for (int i = 0; i < 128; i += 2) {
+                        const unsigned long long z = at_mul2(at_pack2(__uint_as_float(sv[i]), __uint_as_float(sv[i + 1])), zz);
+                        const unsigned long long y = at_mul2(z, z);
+                        unsigned long long p = at_pack2(tc[7], tc[7]);
+#pragma unroll
+                        for (int c = 6; c >= 0; --c) p = at_fma2(p, y, at_pack2(tc[c], tc[c]));
+                        p = at_mul2(p, z);
+                        sv[i] = __float_as_uint(at_lo(p));
+                        sv[i + 1] = __float_as_uint(at_hi(p));
+                    }
+                } else {
+                    const float k2 = 2.f * log2e * z_of;      // tanh(z) = 1 - 2 / (1 + 2^(2 z log2 e))
+#pragma unroll
+                    for (int i = 0; i < 128; ++i) {
+                        float e, q;
+                        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(__uint_as_float(sv[i]) * k2));
+                        asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(q) : "f"(1.f + e));
+                        sv[i] = __float_as_uint(fmaf(-2.f, q, 1.f));
+                    }
+                }
+            }
             if (edge) {
 #pragma unroll
                 for (int i = 0; i < 128; ++i)
                     if (kbase + i > qpos) sv[i] = 0xff800000u;      // -inf: not visible
+            }
+            if (EXT && kbase < low_last) {
+#pragma unroll
+                for (int i = 0; i < 128; ++i)
+                    if (kbase + i < low) sv[i] = 0xff800000u;
             }
             float tmax = -INFINITY, tmax2 = -INFINITY;
 #pragma unroll
@@ -382,7 +477,7 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             unsigned long long psum2 = 0ull, psum2b = 0ull;
 #pragma unroll
             for (int c = 0; c < 4; ++c) {
-                unsigned pk[16];
+                unsigned pk[16], pr[EXT ? 16 : 1];
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
                     unsigned long long x2;
@@ -394,8 +489,14 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                     else asm("add.rn.f32x2 %0, %1, %2;" : "=l"(psum2) : "l"(psum2), "l"(at_pack2(e0, e1)));
                     __nv_bfloat162 bb = __floats2bfloat162_rn(e0, e1);
                     pk[i >> 1] = *reinterpret_cast<unsigned*>(&bb);
+                    if (EXT) {
+                        const float2 f = __bfloat1622float2(bb);
+                        __nv_bfloat162 rr = __floats2bfloat162_rn(e0 - f.x, e1 - f.y);
+                        pr[EXT ? i >> 1 : 0] = *reinterpret_cast<unsigned*>(&rr);
+                    }
                 }
                 AT_ST16(pk, tmem_s + lane_addr + (unsigned)(16 * c));
+                if constexpr (EXT) AT_ST16(pr, tmem_s + lane_addr + (unsigned)(64 + 16 * c));
             }
             asm("add.rn.f32x2 %0, %1, %2;" : "=l"(psum2) : "l"(psum2), "l"(psum2b));
             l_run = l_run * corr + (at_lo(psum2) + at_hi(psum2));
@@ -417,6 +518,17 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
                 unsigned ov[32];
                 AT_LD32(ov, tmem_o + lane_addr + c0);
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+                if (EXT && ext.gate_logits && row < rows_valid) {
+                    const float4* gl = reinterpret_cast<const float4*>(ext.gate_logits + (size_t)(t0 + row) * ext.ld_gate + (size_t)h * HD + c0);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {
+                        const float4 g = gl[i];
+                        ov[4 * i] = __float_as_uint(__fdividef(__uint_as_float(ov[4 * i]), 1.f + __expf(-g.x)));
+                        ov[4 * i + 1] = __float_as_uint(__fdividef(__uint_as_float(ov[4 * i + 1]), 1.f + __expf(-g.y)));
+                        ov[4 * i + 2] = __float_as_uint(__fdividef(__uint_as_float(ov[4 * i + 2]), 1.f + __expf(-g.z)));
+                        ov[4 * i + 3] = __float_as_uint(__fdividef(__uint_as_float(ov[4 * i + 3]), 1.f + __expf(-g.w)));
+                    }
+                }
                 if (row < rows_valid) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
@@ -877,10 +989,32 @@ static int launch_prefill_tc(const void* q, const void* k_pages, const void* v_p
     if (rc) return rc;
     rc = tc_make_map_rows8(&mv, v_pages, rows, HD / 64, P / 8);
     if (rc) return rc;
-    cudaFuncSetAttribute(paged_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, AtSmem<HD>::bytes);
-    paged_prefill_tc_kernel<HD><<<dim3(H, n_tiles), AT_THREADS, AtSmem<HD>::bytes, stream>>>(
+    auto kern = paged_prefill_tc_kernel<HD, false>;
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, AtSmem<HD>::bytes);
+    kern<<<dim3(H, n_tiles), AT_THREADS, AtSmem<HD>::bytes, stream>>>(
         mq, mk, mv, (bf16*)out, tiles, n_tiles, q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, H, K,
-        scale, err);
+        scale, err, AtExt());
+    AIE_LAUNCH_CHECK();
+}
+
+// the extended form over rows of one plane: a key of HD elements and, unless `tied`, a value of HD behind it
+template <int HD>
+static int launch_prefill_tc_rows(const void* q, const void* pages, void* out, const int* tiles, int n_tiles,
+                                  const int* q_start, const int* q_len, const int* ctx_len, const int* block_table,
+                                  int bt_width, int num_pages, int P, int T, int H, int K, int tied, float scale,
+                                  const AtExt& ext, unsigned* err, cudaStream_t stream) {
+    CUtensorMap mq, mk, mv;
+    int rc = tc_make_map_2d(&mq, q, (unsigned long long)T, (unsigned long long)H * HD, (unsigned long long)H * HD * 2, AT_M, 64);
+    if (rc) return rc;
+    const unsigned long long rows = (unsigned long long)num_pages * K * P, bytes = (unsigned long long)HD * 2 * (tied ? 1 : 2);
+    rc = tc_make_map_rows8(&mk, pages, rows, HD / 64, P / 8, bytes);
+    if (rc) return rc;
+    rc = tc_make_map_rows8(&mv, (const bf16*)pages + (tied ? 0 : HD), rows, HD / 64, P / 8, bytes);
+    if (rc) return rc;
+    auto kern = paged_prefill_tc_kernel<HD, true>;
+    cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, AtSmem<HD>::bytes);
+    launch_pdl(kern, dim3(H, n_tiles), dim3(AT_THREADS), AtSmem<HD>::bytes, stream, mq, mk, mv, (bf16*)out, tiles, n_tiles,
+               q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, H, K, scale, err, ext);
     AIE_LAUNCH_CHECK();
 }
 
@@ -900,6 +1034,27 @@ extern "C" int aie_paged_attention_prefill_tc(const void* q, const void* k_pages
 #define ARGS q, k_pages, v_pages, out, tiles, n_tiles, q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, T, H, K, \
              scale, err, stream
     return d == 128 ? launch_prefill_tc<128>(ARGS) : launch_prefill_tc<64>(ARGS);
+#undef ARGS
+}
+
+// The extended form (see the head of this file) over pages [num_pages, K, P, 2 d] of rows [k | v], or with `tied`
+// [num_pages, K, P, d] of rows that are key and value at once.  window 0: every earlier key; cap 0: unbounded scores;
+// gate_logits [T, >= H d] float32 with rows ld_gate apart, or null.  Same sizes as above.
+extern "C" int aie_paged_attention_prefill_tc_rows(const void* q, const void* pages, void* out, const int* tiles,
+                                                   int n_tiles, const int* q_start, const int* q_len, const int* ctx_len,
+                                                   const int* block_table, int bt_width, int num_pages, int P, int T,
+                                                   int H, int K, int d, int window, int tied, float cap,
+                                                   const float* gate_logits, int ld_gate, float scale, unsigned* err,
+                                                   cudaStream_t stream) {
+    if (n_tiles <= 0) return 0;
+    if (K <= 0 || H % K || window < 0 || cap < 0.f) return AIE_BAD_ARG;
+    if ((d != 64 && d != 128) || P < 8 || P > 128 || 128 % P || n_tiles > 65535) return AIE_UNSUPPORTED;
+    if (((size_t)q & 15) || ((size_t)pages & 15) || ((size_t)out & 15)) return AIE_UNSUPPORTED;
+    if (gate_logits && (((size_t)gate_logits & 15) || ld_gate % 4)) return AIE_UNSUPPORTED;
+    const AtExt ext{window, cap, gate_logits, ld_gate};
+#define ARGS q, pages, out, tiles, n_tiles, q_start, q_len, ctx_len, block_table, bt_width, num_pages, P, T, H, K, tied, \
+             scale, ext, err, stream
+    return d == 128 ? launch_prefill_tc_rows<128>(ARGS) : launch_prefill_tc_rows<64>(ARGS);
 #undef ARGS
 }
 

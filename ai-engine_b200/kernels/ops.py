@@ -574,6 +574,31 @@ def paged_attention_prefill_tc(q, k_pages, v_pages, tiles, q_start, q_len, ctx_l
     return True
 
 
+def paged_attention_prefill_rows(q, pages, work, ctx, block_table, scale: float, window: int, softcap: float, tied: bool,
+                                 gate_logits, out, cost=(0.0, 0.0)) -> bool:
+    """The tcgen05 prompt kernel over cache rows [k | v] of one plane (`tied`: rows that are key and value at once), with a
+    window, bounded scores, a sigmoid gate on every output element, and probabilities that meet the values as two bfloat16
+    terms.  q, out [T, H, d] bfloat16; gate_logits a float32 view [T, H * d] or None.  False (nothing was launched) for
+    sizes it does not take: keys and values of one size other than 64 or 128, pages that do not divide 128 or hold fewer
+    than 8 keys, a gate whose rows do not start on 16 bytes."""
+    T, H, d = q.shape
+    num_pages, K, P, w = pages.shape
+    if d not in (64, 128) or out.shape[2] != d or P < 8 or P > 128 or 128 % P:
+        return False
+    if gate_logits is not None and (gate_logits.stride(0) % 4 or gate_logits.data_ptr() % 16):
+        return False
+    _dev(q, pages, out, block_table, work.prefill_tiles)
+    tiles = work.prefill_tiles
+    with region("attention_prefill_tcgen05", *cost):
+        check(library("attention_prefill_tc.cu").aie_paged_attention_prefill_tc_rows(
+            _p(q), _p(pages), _p(out), _p(tiles), c_int(tiles.shape[0]), _p(ctx.q_start), _p(ctx.q_len), _p(ctx.ctx_len),
+            _p(block_table), c_int(block_table.shape[1]), c_int(num_pages), c_int(P), c_int(T), c_int(H), c_int(K), c_int(d),
+            c_int(window), c_int(1 if tied else 0), c_float(softcap), _p(gate_logits),
+            c_int(gate_logits.stride(0) if gate_logits is not None else 0), c_float(scale), _p(ctx.err), _stream()),
+            "paged_attention_prefill_tc_rows")
+    return True
+
+
 def prefill_takes_pairs(n_tiles: int, n_units: int, heads: int) -> bool:
     """Whether the tcgen05 prompt kernel with two query tiles per CTA is the faster one for a step with `n_tiles`
     tiles in `n_units` units of two.  Measured on heads of 128 and of 64: it takes 0.80-0.86 of the one-tile
@@ -1263,7 +1288,9 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
     softcap c > 0: the scaled product is replaced by c * tanh(it / c).  gate_logits: a float32 view [T, H * e] with any
     row stride; every output element is multiplied by its sigmoid.  tied: values are the keys, a row is that one vector.
     bfloat16 with the sizes of `sink_attention_fast`: lone tokens take the split-KV kernel, portions of prompts
-    the tiled tensor-core kernel (`work`: the attention work lists); everything else takes the plain kernel."""
+    the tcgen05 kernel where the layer has nothing that it does not know (a sink, a bias, kept keys, chunks, several maps)
+    and sizes that it takes, else the tiled mma.sync kernel (`work`: the attention work lists); everything else takes the
+    plain kernel."""
     _dev(q, pages, gate, temp, slope, sink, block_table)
     T, H, d = q.shape
     G = pages.shape[1]
@@ -1314,6 +1341,11 @@ def sink_attention(q: torch.Tensor, pages: torch.Tensor, gate: Optional[torch.Te
         if work.n_decode < ctx.R:
             tiles = work.prefill_tiles
             share = 1.0 - float(work.n_decode) / T
+            plain_rows = (gate is None and temp is None and slope is None and sink is None and not keep_first and not chunk
+                          and maps == 1 and d == e and out32 is None)
+            if plain_rows and paged_attention_prefill_rows(q, pages, work, ctx, block_table, scale, window, softcap, tied,
+                                                           gate_logits, out, (cost[0] * share, cost[1] * share)):
+                return out
             with region("sink_attention_prefill", cost[0] * share, cost[1] * share):
                 check(fast.aie_sink_attention_prefill(_p(q), _p(pages), _p(out), _p(gate), _p(temp), _p(slope), _p(sink),
                                                       _p(tiles), c_int(tiles.shape[0]), _p(ctx.q_start), _p(ctx.q_len),

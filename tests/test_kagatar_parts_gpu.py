@@ -146,14 +146,21 @@ def test_attention_three_requests_in_unequal_portions(dtype, shape):
     rig.cache.book.check_invariants()
 
 
-KINDS = {      # by kind and whether the sizes take the tensor-core kernels in bfloat16; the window is put in by the test
-    "tied": lambda d: tied(4, 4, d, 0.35), "gated": lambda d: gated(4, 2, d, 40, 0.35, rot(1e4, 4, yarn(4.0, 200))),
-    "capped": lambda d: capped(4, 2, d, 24, 3.0, rot(1e4, 4, waves(4.0, 200)), None, 30.0)}
+def value_size(d, other):
+    """Keys and values of 64 or of 128 take the tcgen05 prompt kernel in bfloat16, other sizes the mma.sync or the plain one."""
+    return d if d in (64, 128) else other
+
+
+KINDS = {      # the window is put in by the test
+    "tied": lambda d: tied(4, 4, d, 0.35),
+    "gated": lambda d: gated(4, 2, d, value_size(d, 40), 0.35, rot(1e4, 4, yarn(4.0, 200))),
+    "capped": lambda d: capped(4, 2, d, value_size(d, 24), 36.0 / d, rot(1e4, 4, waves(4.0, 200)), None, 30.0)}
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("kind", sorted(KINDS))
-@pytest.mark.parametrize("dim,window,page", [(30, 40, 8), (32, 40, 8), (40, 90, 16), (64, 130, 32), (128, 65, 8), (32, 0, 8)])
+@pytest.mark.parametrize("dim,window,page", [(30, 40, 8), (32, 40, 8), (40, 90, 16), (64, 130, 32), (128, 65, 8), (32, 0, 8),
+                                             (64, 0, 64), (128, 200, 32), (64, 33, 8)])
 def test_planted_keys_at_every_edge(dtype, kind, dim, window, page):
     """Pairs of tokens with a strong input that the later one's query and the earlier one's key read alike, so that the
     later one's weight goes to the earlier one when it reads it: just inside the window and just outside, at a page's
@@ -189,12 +196,12 @@ def test_planted_keys_at_every_edge(dtype, kind, dim, window, page):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("dim", [30, 32, 72])
+@pytest.mark.parametrize("dim", [30, 32, 72, 64, 128])
 def test_scores_at_their_bound(dtype, dim):
     """Scores many times the bound: the weights are those of +-softcap, far from a softmax without it, in prompts and for
     single tokens; and a bound far above the scores changes nothing."""
     gen = torch.Generator().manual_seed(dim)
-    l = capped(4, 2, dim, 16, 2.0, None, 60, 1.5)
+    l = capped(4, 2, dim, value_size(dim, 16), 2.0, None, 60, 1.5)
     part, t = attention_part(l, 64, 1e-5, dtype, gen)
     h = rnd(gen, 90, 64)
     ref = plain(l, t, h, 1e-5)
@@ -202,10 +209,58 @@ def test_scores_at_their_bound(dtype, dim):
     assert float((loose - ref).abs().max()) > float(ref.std())
     for cuts in ([90], [30] + [1] * 60):
         near(Rig(part, DT[dtype], page=8).run([h.to(DT[dtype])], [cuts])[0], ref, dtype, f"bounded scores {cuts[:2]}")
-    l = capped(4, 2, dim, 16, 0.1, None, 60, 1e4)
+    l = capped(4, 2, dim, value_size(dim, 16), 0.1, None, 60, 1e4)
     part, t = attention_part(l, 64, 1e-5, dtype, gen)
     free = plain(dict(l, mixer=dict(l["mixer"], softcap=None)), t, h, 1e-5)
     near(Rig(part, DT[dtype], page=8).run([h.to(DT[dtype])], [[40] + [1] * 50])[0], free, dtype, "a bound out of reach")
+
+
+@pytest.mark.parametrize("d,window,page,tied_values,cap,spread,gate", [
+    (64, 0, 16, False, 0.0, 1.0, True), (128, 150, 16, False, 30.0, 8.0, False), (128, 70, 8, True, 0.0, 1.0, False),
+    (64, 129, 32, True, 4.0, 6.0, True), (128, 0, 128, False, 5.0, 40.0, True), (64, 1, 8, False, 20.0, 2.0, False),
+    (64, 300, 64, False, 1e3, 1.0, True)])
+def test_three_prompt_kernels_agree(monkeypatch, d, window, page, tied_values, cap, spread, gate):
+    """bfloat16 queries and cache rows through the tcgen05, the mma.sync and the plain kernel: portions that start inside
+    a page, at its edge and far in, whose early pages the window has given back; scores under and far over the bound
+    (both forms of its tanh)."""
+    from ai_engine_b200.cache import PagedCache
+    from ai_engine_b200.engine.step import StepContext, StepEntry
+    from ai_engine_b200.kernels import ops
+    from ai_engine_b200.parts import ATTENTION_WORK, CacheNeed, KVRequest
+    gen = torch.Generator().manual_seed(d + window + page)
+    H, G, w = 6, 2, d if tied_values else 2 * d
+    cache = PagedCache([CacheNeed(0, "p", KVRequest(G, w, window, planes=1))], page, 2048 // page, 3, 1024, torch.bfloat16, DEV)
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+    entries = []
+    for have, n in ((0, 190), (page, 129), (517, 140)):
+        slot = cache.admit()
+        assert cache.ensure(slot, have + n)
+        cache.advance(slot, have)
+        entries.append(StepEntry(slot, have, [0] * n, []))
+    ctx = StepContext(entries, cache, torch.device(DEV), err, planners=(ATTENTION_WORK,))
+    lc = cache.part_cache(0, "p", ctx)
+    T = ctx.T
+    lc.k_pages.copy_(torch.randn(lc.k_pages.shape, generator=gen).to(DEV))
+    for r, e in enumerate(entries):              # a place that no token has written yet holds no number
+        for p in range(e.start + len(e.tokens), -(-(e.start + len(e.tokens)) // page) * page):
+            lc.k_pages[int(lc.block_table[r, p // page]), :, p % page] = float("nan")
+    q = (torch.randn(T, H, d, generator=gen) * spread).to(DEV).to(torch.bfloat16)
+    logits = torch.randn(T, H * d + 12, generator=gen).to(DEV)[:, 8:8 + H * d] if gate else None
+    go = lambda: ops.sink_attention(q, lc.k_pages, None, None, None, None, ctx, ctx.plan(ATTENTION_WORK), lc.block_table, d,
+                                    d ** -0.5, window, 0, softcap=cap, tied=tied_values, gate_logits=logits).float().cpu()
+    calls = []
+    real = ops.paged_attention_prefill_rows
+    monkeypatch.setattr(ops, "paged_attention_prefill_rows", lambda *a, **k: calls.append(real(*a, **k)) or calls[-1])
+    tc = go()
+    assert calls == [True]
+    monkeypatch.setattr(ops, "paged_attention_prefill_rows", lambda *a, **k: False)
+    mma = go()
+    monkeypatch.setattr(ops, "sink_attention_fast", lambda *a, **k: False)
+    ref = go()
+    assert int(err.item()) == 0 and bool(torch.isfinite(ref).all())
+    for name, got in (("tcgen05", tc), ("mma.sync", mma)):
+        assert float((got - ref).abs().max()) <= 6e-3 * float(ref.abs().max()), name       # one rounding to bfloat16
+        assert float((got - ref).abs().mean()) <= 2e-4 * float(ref.abs().max()), name
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
